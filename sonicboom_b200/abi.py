@@ -49,11 +49,13 @@ CORE = {
     "sb_glu_clamped": ("i", "piiffipis"),
     "sb_gated_act": ("i", "piiiffipis"),
     "sb_scale": ("i", "pzfs"),
+    "sb_stream_join": ("i", "ppiipiifpippifpis"),
+    "sb_side_gate": ("i", "piiippiiiipis"),
     "sb_latent_prep": ("i", "piiiiiipppppipifpipiiipiifs"),
     "sb_head_linear": ("i", "pizzpiiiiipizzs"),
     "sb_mlstm_scan": ("i", "pippiiippiffipipps"),
     "sb_mlstm_out": ("i", "pppiiiipifpis"),
-    "sb_attention_plain": ("i", "ppiippppipiiiiifpfs"),
+    "sb_attention_plain": ("i", "ppiippppipiiiiifpfipis"),
     "sb_stream_add": ("i", "pppiiippifpis"),
     "sb_polynorm": ("i", "piipifpis"),
     "sb_attn_prep": ("i", "piiiiiiiiiiiippppiiffppppipipiis"),
@@ -64,21 +66,24 @@ CORE = {
     "sb_linrec_out": ("i", "ppiiiiipiiifpis"),
     "sb_embed_pair": ("i", "pippppppiipiiiifps"),
     "sb_keep_last_token": ("i", "pppips"),
-    "sb_layernorm": ("i", "ppiipifpis"),
+    "sb_layernorm": ("i", "ppiippifpis"),
     "sb_causal_conv": ("i", "piiiiippiiiipppppppiiis"),
+    "sb_conv_heads": ("i", "piiiiiiiipiipppppppipppis"),
+    "sb_conv_heads_max_taps": ("i", ""),
     "sb_delta_prep": ("i", "piiiiiiiipppiffps"),
     "sb_delta_scan": ("i", "piiiipippiipps"),
     "sb_ssd_prep": ("i", "piiipiiiiippips"),
     "sb_ssd_out": ("i", "ppiiipiiiiippifpis"),
     "sb_attention_sigmoid": ("i", "ppiippiippppipiiiiiiffps"),
     "sb_moe_route": ("i", "piiipps"),
-    "sb_moe_route_scored": ("i", "ppiiiiiifipps"),
+    "sb_moe_route_scored": ("i", "pipiiiiiiifipps"),
     "sb_moe_tile_rows": ("i", "iiiii"),
     "sb_moe_max_tiles": ("i", "iii"),
     "sb_moe_group": ("i", "piiipps"),
-    "sb_moe_up": ("i", "pipippiiiiiiffps"),
+    "sb_moe_up": ("i", "pipippiiiiiiiffps"),
     "sb_moe_down": ("i", "pipippiiiiiips"),
     "sb_moe_combine": ("i", "pppiiis"),
+    "sb_moe_join": ("i", "ppppipippipiiiipis"),
     "sb_sample_params_size": ("i", ""),
     "sb_sample": ("i", "piippipps"),
     "sb_add_i32": ("i", "piis"),
@@ -91,7 +96,7 @@ ATTENTION = {
     "sb_attention_status": ("i", ""),
     "sb_attention_last_launches": ("i", ""),
     "sb_attention_scratch_bytes": ("z", "iiiii"),
-    "sb_attention": ("i", "ppiiippppipiiiifpzpiiiipzpfs"),
+    "sb_attention": ("i", "ppiiippppipiiiifpzpiiiipzpfipis"),
     "sb_attention_decode_static": ("i", "ppiiippppipiiiifis"),
     "sb_attention_static_scratch_bytes": ("z", ""),
 }

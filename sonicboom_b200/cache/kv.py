@@ -11,7 +11,8 @@ at a time; here sequences of a batch share pools of pages.
   pool of pages, one page list per sequence (all entries of a group grow together).
 * A group with a window gives back the pages whose keys no later query can see, so a
   sequence holds about `window` keys there, however long it grows (plus the pages of the first
-  `keep_first` keys, when the window keeps those in sight for good).
+  `keep_first` keys, when the window keeps those in sight for good).  A group whose queries see their own
+  chunk of positions only gives back the pages of the chunks before it.
 * A **slot** is a sequence's record: its length, its page lists, and its row in every state
   tensor.  A schedule entry may ask for one state tensor or for several by name; the model as a
   whole may ask for named ones too (`model_state`).  `state` maps an entry's index, or (entry,
@@ -38,6 +39,12 @@ class KVNeed:
     head_dim: int
     window: int = 0            # 0: all keys stay; n: only the last n keys are ever read
     keep_first: int = 0        # with a window: the first n keys of a sequence are read for good too
+    chunk: int = 0             # n: only keys of the query's own stretch of n positions (from position 0) are read
+
+    def first_read(self, pos: int) -> int:
+        """The first key, kept first ones aside, that a query at position `pos` or later reads."""
+        lo = max(0, pos - self.window + 1) if self.window > 0 else 0
+        return max(lo, pos // self.chunk * self.chunk) if self.chunk > 0 else lo
 
 
 @dataclass(frozen=True)
@@ -176,11 +183,10 @@ class Cache:
             raise CacheError(f"slot {slot}: advance to {new_len} without pages for it")
         rec.length = new_len
         for g, pages in zip(self.groups, rec.pages):
-            w = g.need.window
-            if w <= 0:
+            if g.need.window <= 0 and g.need.chunk <= 0:
                 continue
-            # the next query sits at position >= new_len and sees keys j > position - w
-            dead_pages = max(0, new_len - w + 1) // self.page_size     # pages wholly at j <= new_len - w
+            # the next query sits at position >= new_len: pages wholly before what it reads are dead
+            dead_pages = g.need.first_read(new_len) // self.page_size
             kept_pages = (g.need.keep_first + self.page_size - 1) // self.page_size   # pages with a key that stays in sight
             dead = range(kept_pages, min(dead_pages, len(pages)))
             give = [pages[i] for i in dead if pages[i] is not None]
@@ -201,7 +207,7 @@ class Cache:
             return False         # fixed-size state has moved on with the tokens and cannot go back
         keep = (new_len + self.page_size - 1) // self.page_size
         for g, pages in zip(self.groups, rec.pages):
-            first_seen = max(0, new_len - g.need.window + 1) // self.page_size if g.need.window else 0
+            first_seen = g.need.first_read(new_len) // self.page_size
             if any(p is None for p in pages[first_seen:keep]):      # (pages of kept first keys are never given back)
                 return False
         for g, pages in zip(self.groups, rec.pages):

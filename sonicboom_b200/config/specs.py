@@ -33,6 +33,7 @@ class NormSpec:
     width: int
     eps: float
     tensor: str                    # tensor name of the weight
+    bias: Optional[str] = None     # tensor name of the bias, for kinds that have one
 
 
 @dataclass(frozen=True)
@@ -84,6 +85,27 @@ class PairEmbeddingSpec:
 
 
 @dataclass(frozen=True)
+class SideTableSpec:
+    """A second embedding table whose rows hold one part of `dim` values for every layer that takes a
+    token input of its own.  `tensor` is [vocab, parts * dim]."""
+    tensor: str
+    dim: int
+    parts: int
+
+
+@dataclass(frozen=True)
+class SideInputSpec:
+    """What a layer makes of its part of the side table, added to the stream after its feed-forward:
+    g = gelu(gate x) * e, y = proj g, x + y / sqrt(mean(y^2) + eps) * norm.  `part` numbers the layer's
+    part; the tensors are `prefix` + gate [dim, width], proj [width, dim], norm [width]."""
+    prefix: str
+    width: int
+    dim: int
+    part: int
+    eps: float
+
+
+@dataclass(frozen=True)
 class DepthMixSpec:
     """What goes on to the next schedule entry instead of a block's own result: a combination of
     the embedding output and every block result so far (`n_inputs` of them, this block's last)."""
@@ -107,6 +129,9 @@ class LayerSpec:
     depth_mix: Optional[DepthMixSpec] = None
     mixer_conv: Optional[ConvSpec] = None          # on the mixer's input, after its norm
     feed_forward_conv: Optional[ConvSpec] = None   # on the feed-forward's input, after its norm
+    mixer_scale: Optional[str] = None              # tensor [width] that multiplies the mixer's result channel by channel
+    feed_forward_scale: Optional[str] = None       # the same for the feed-forward's
+    side_input: Optional[SideInputSpec] = None     # the layer's token input, after the feed-forward
     params: tuple = ()             # extra (key, value) pairs for arrangements with constants of their own
 
     @property
@@ -152,6 +177,7 @@ class ModelSpec:
     injections: tuple = ()              # of StreamInjection, at most one per schedule entry
     unused_tensors: tuple = ()          # (name, shape) of tensors a file may hold that nothing reads
     pair_embedding: Optional[PairEmbeddingSpec] = None   # added to every embedding row
+    side_table: Optional[SideTableSpec] = None           # read by the layers that have a side input
 
     def validate(self) -> None:
         if not self.layers:
@@ -162,6 +188,12 @@ class ModelSpec:
             raise ConfigError(f"logit_scale {self.logit_scale} must be positive")
         if self.logit_cap < 0.0:
             raise ConfigError(f"logit_cap {self.logit_cap} must be zero (none) or positive")
+        for i, l in enumerate(self.layers):
+            side = l.side_input
+            if side is not None and (self.side_table is None or side.dim != self.side_table.dim
+                                     or not 0 <= side.part < self.side_table.parts):
+                raise ConfigError(f"layer {i} reads part {side.part} of {side.dim} values of a side table that the "
+                                  f"model does not have ({self.side_table})")
         seen = set()
         for inj in self.injections:
             if not 0 <= inj.before_entry < len(self.schedule) or inj.before_entry in seen:

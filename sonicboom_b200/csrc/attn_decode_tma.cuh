@@ -85,8 +85,9 @@ __device__ __forceinline__ uint32_t dt_addr(uint32_t tile, int row, int chunk) {
 }
 
 // One warp's 32 keys (rows key_row0 ... + 31 of the tile) for its 16 query rows.
+template <bool BIAS>
 __device__ __forceinline__ void dt_tile_step(uint32_t qs, uint32_t ks, uint32_t vs,
-                                             int key_row0, int key0, int pos_a, int pos_b, int window,
+                                             int key_row0, int key0, const RowView& ra, const RowView& rb, int bias_last,
                                              const ScoreMap sm, float (&m)[2], float (&l)[2],
                                              float (&o)[HD / 8][4], int lane) {
   float s[4][4];
@@ -116,9 +117,9 @@ __device__ __forceinline__ void dt_tile_step(uint32_t qs, uint32_t ks, uint32_t 
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const int key = key0 + j * 8 + 2 * t + (i & 1);
-      const int pos = (i < 2) ? pos_a : pos_b;
-      const bool seen = key <= pos && (window == 0 || pos - key < window);
-      const float v = seen ? mapped_score(s[j][i], sm) : -INFINITY;
+      const RowView& rv = (i < 2) ? ra : rb;
+      const bool seen = key <= rv.pos && key >= rv.lo;
+      const float v = seen ? row_score<BIAS>(s[j][i], sm, rv, key, bias_last) : -INFINITY;
       s[j][i] = v;
       tmax[i >> 1] = fmaxf(tmax[i >> 1], v);
     }
@@ -192,7 +193,7 @@ __device__ __forceinline__ bool dt_item(const AttnParams& p, int item, DtItem& i
   it.pos0 = p.seq_pos0[it.b];
   it.R = n_new * G;
   it.p_hi = it.pos0 + n_new - 1;
-  const int key_lo = p.window > 0 ? max(0, it.pos0 - p.window + 1) : 0;
+  const int key_lo = low_key(p, max(it.pos0, 0));
   const int sp = split_pages_for(it.p_hi + 1);
   it.split_lo = key_lo / (sp * KT);
   it.split_hi = it.p_hi / (sp * KT);
@@ -232,7 +233,7 @@ __global__ void __launch_bounds__(DT_MERGE_THREADS) attn_merge_kernel(const Attn
   const int G = p.n_q_heads / p.n_kv_heads;
   const int row0 = p.seq_row0[b], n_new = p.seq_row0[b + 1] - row0, pos0 = p.seq_pos0[b];
   const int R = n_new * G, p_hi = pos0 + n_new - 1;
-  const int key_lo = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
+  const int key_lo = low_key(p, max(pos0, 0));
   const int sp = split_pages_for(p_hi + 1);
   const int split_lo = key_lo / (sp * KT), split_hi = p_hi / (sp * KT);
   // one split, or a sequence the attention kernel gave rows of zeros: nothing to merge
@@ -312,6 +313,7 @@ __global__ void __launch_bounds__(DT_MERGE_THREADS) attn_merge_kernel(const Attn
   }
 }
 
+template <bool BIAS>
 __global__ void __launch_bounds__(DT_THREADS, DT_BLOCKS_PER_SM)
 attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_kv, const AttnParams p, int n_items) {
   extern __shared__ __align__(1024) unsigned char dt_smem[];
@@ -484,7 +486,8 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_kv, const AttnPar
       // item left: their results are never written); thread 0 saw the copy complete
       mbar_wait(qfull0 + 8 * d, ((k - 1) / DT_QUEUE) & 1, 26);
       const uint32_t qs = q_s + d * DT_Q_BYTES;
-      const int pos_a = ra < w.R ? w.pos0 + ra / G : -1, pos_b = rb < w.R ? w.pos0 + rb / G : -1;
+      const RowView va = row_view<BIAS>(p, ra < w.R ? w.pos0 + ra / G : -1, w.kvh * G + ra % G);
+      const RowView vb = row_view<BIAS>(p, rb < w.R ? w.pos0 + rb / G : -1, w.kvh * G + rb % G);
       float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f};
       float o[HD / 8][4];
 #pragma unroll
@@ -502,8 +505,8 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_kv, const AttnPar
           continue;
         }
         const uint32_t ks = ring + s * DT_STAGE_BYTES, vs = ks + DT_TILE_BYTES;
-        dt_tile_step(qs, ks, vs, half * 32, (w.tile_lo + j) * KT + half * 32, pos_a, pos_b, p.window,
-                     score_map(p), m, l, o, lane);
+        dt_tile_step<BIAS>(qs, ks, vs, half * 32, (w.tile_lo + j) * KT + half * 32, va, vb, p.bias_len - 1,
+                           score_map(p), m, l, o, lane);
         if (j + 1 < w.n_tiles) {                       // the last tile's stage stays for the merge
           __syncwarp();
           if (lane == 0) mbar_arrive(empty0 + 8 * s);
@@ -577,6 +580,20 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_kv, const AttnPar
       if (pair == last_pair && lane == 0) mbar_arrive(empty0 + 8 * s_merge);
     }
   }
+}
+
+template <bool BIAS>
+int configure_decode_tma() {
+  static bool configured = false;
+  if (configured) return SB_OK;
+  cudaError_t e = cudaFuncSetAttribute(attn_decode_tma_kernel<BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize, DT_SMEM);
+  if (e == cudaSuccess)                          // all of the SM's memory as shared memory: three blocks fit
+    e = cudaFuncSetAttribute(attn_decode_tma_kernel<BIAS>, cudaFuncAttributePreferredSharedMemoryCarveout,
+                             cudaSharedmemCarveoutMaxShared);
+  if (e != cudaSuccess)
+    SB_FAIL(SB_ERR_CUDA, "sb_attention: shared memory opt-in failed: %s", cudaGetErrorString(e));
+  configured = true;
+  return SB_OK;
 }
 
 }  // namespace

@@ -23,8 +23,12 @@
 //    on where the pages lie.
 //
 // Mask: key j is visible to the query at position i when j <= i and (window == 0 or
-// i - j < window) (core/src/nn/attention.cpp:66-70).  The scale multiplies the finished dot
-// product in float32.  Probabilities are rounded to bfloat16 only as the P.V operand.
+// i - j < window) (core/src/nn/attention.cpp:66-70); with a chunk size c > 0 also only when j lies
+// in the query's own chunk, floor(j / c) = floor(i / c).  Both are a lowest visible key that grows
+// with i (low_key).  The scale multiplies the finished dot product in float32.  With a distance
+// bias (`bias` [n_q_heads][bias_len]) the finished, capped score gets bias[h][min(i - j, bias_len - 1)]
+// added; the kernels that do so are instantiations of their own (BIAS), so that others carry
+// nothing of it.  Probabilities are rounded to bfloat16 only as the P.V operand.
 #include <math.h>
 
 #include "common.cuh"
@@ -64,9 +68,12 @@ struct AttnParams {
   float* scratch;
   int* counters;               // one per (sequence, key/value head), zero between launches
   int n_q_heads, n_kv_heads, window, n_splits;
+  int chunk;                   // > 0: keys of the query's own stretch of this many positions only
   int n_seqs;
   float scale_log2;            // scale * log2(e)
   float cap_a, cap_b;          // a score cap c > 0: cap_a = scale / c, cap_b = c log2(e); else both 0
+  const float* bias;           // [n_q_heads][bias_len] by distance, the last one for all larger ones (or null)
+  int bias_len;
   const float* sink;           // [n_q_heads] or null: exp(sink) joins each row's softmax denominator
   const char* warm;            // decode: bytes the next kernel will read, asked into L2 (or null)
   size_t warm_bytes;
@@ -91,6 +98,27 @@ __device__ __forceinline__ float mapped_score(float dot, const ScoreMap& sm) {
 }
 __device__ __forceinline__ ScoreMap score_map(const AttnParams& p) {
   return ScoreMap{p.scale_log2, p.cap_a, p.cap_b};
+}
+// The first key that the query at position `pos` sees.
+__device__ __forceinline__ int low_key(const AttnParams& p, int pos) {
+  const int w = p.window > 0 ? max(0, pos - p.window + 1) : 0;
+  return p.chunk > 0 ? max(w, pos / p.chunk * p.chunk) : w;
+}
+// What a thread needs to know of one of its query rows: the row's position (-1: a padding row, which
+// sees nothing), its first visible key, and its head's row of the distance bias.
+struct RowView {
+  int pos, lo;
+  const float* bias;
+};
+template <bool BIAS>
+__device__ __forceinline__ RowView row_view(const AttnParams& p, int pos, int head) {
+  return RowView{pos, low_key(p, max(pos, 0)), BIAS ? p.bias + (size_t)head * p.bias_len : nullptr};
+}
+// The exponent's argument of one visible key's score, with the row's distance bias.
+template <bool BIAS>
+__device__ __forceinline__ float row_score(float dot, const ScoreMap& sm, const RowView& rv, int key, int bias_last) {
+  const float v = mapped_score(dot, sm);
+  return BIAS ? fmaf(__ldg(rv.bias + min(max(rv.pos - key, 0), bias_last)), LOG2E, v) : v;
 }
 
 __device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0,
@@ -141,11 +169,11 @@ __device__ __forceinline__ void load_kv_tile(uint32_t ks, uint32_t vs, const bf1
 }
 
 // One key tile for a warp's 16 rows: scores, mask, online softmax update, P.V.
-// `pos_a`, `pos_b`: positions of the thread's two rows (g and g + 8), -1 for padding rows.
-template <int NKEYS>
+// `ra`, `rb`: the thread's two rows (g and g + 8).
+template <int NKEYS, bool BIAS>
 __device__ __forceinline__ void tile_step(const uint32_t (&qf)[HD / 16][4], uint32_t ks,
-                                          uint32_t vs, int key0, int pos_a, int pos_b, int window,
-                                          const ScoreMap sm, float (&m)[2], float (&l)[2],
+                                          uint32_t vs, int key0, const RowView& ra, const RowView& rb,
+                                          int bias_last, const ScoreMap sm, float (&m)[2], float (&l)[2],
                                           float (&o)[HD / 8][4], int lane) {
   float s[NKEYS / 8][4];
 #pragma unroll
@@ -171,9 +199,9 @@ __device__ __forceinline__ void tile_step(const uint32_t (&qf)[HD / 16][4], uint
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const int key = key0 + j * 8 + 2 * t + (i & 1);
-      const int pos = (i < 2) ? pos_a : pos_b;
-      const bool seen = key <= pos && (window == 0 || pos - key < window);
-      const float v = seen ? mapped_score(s[j][i], sm) : -INFINITY;
+      const RowView& rv = (i < 2) ? ra : rb;
+      const bool seen = key <= rv.pos && key >= rv.lo;
+      const float v = seen ? row_score<BIAS>(s[j][i], sm, rv, key, bias_last) : -INFINITY;
       s[j][i] = v;
       tmax[i >> 1] = fmaxf(tmax[i >> 1], v);
     }
@@ -246,6 +274,7 @@ namespace {
 // ------------------------------------------------------------------------------- prefill
 constexpr int PREFILL_SMEM = (BM + 4 * KT) * LDS * 2;
 
+template <bool BIAS>
 __global__ void __launch_bounds__(PREFILL_THREADS) attn_prefill_kernel(const AttnParams p) {
   extern __shared__ __align__(128) unsigned char smem[];
   const uint32_t qs = (uint32_t)__cvta_generic_to_shared(smem);
@@ -275,7 +304,7 @@ __global__ void __launch_bounds__(PREFILL_THREADS) attn_prefill_kernel(const Att
   }
   const int r_last = min(R, r_base + BM) - 1;
   const int p_lo = pos0 + r_base / G, p_hi = pos0 + r_last / G;
-  const int tile_lo = (p.window > 0 ? max(0, p_lo - p.window + 1) : 0) / KT, tile_hi = p_hi / KT;
+  const int tile_lo = low_key(p, p_lo) / KT, tile_hi = p_hi / KT;
   load_kv_tile(kv0, kv0 + KT * LDS * 2, p.cache, pages[tile_lo], p.n_kv_heads, kvh, tid, PREFILL_THREADS);
   cp_async_commit();
   cp_async_wait<0>();
@@ -284,7 +313,8 @@ __global__ void __launch_bounds__(PREFILL_THREADS) attn_prefill_kernel(const Att
   uint32_t qf[HD / 16][4];
   load_q_frags(qs, warp * 16, lane, qf);
   const int ra = r_base + warp * 16 + (lane >> 2), rb = ra + 8;
-  const int pos_a = ra < R ? pos0 + ra / G : -1, pos_b = rb < R ? pos0 + rb / G : -1;
+  const RowView va = row_view<BIAS>(p, ra < R ? pos0 + ra / G : -1, kvh * G + ra % G);
+  const RowView vb = row_view<BIAS>(p, rb < R ? pos0 + rb / G : -1, kvh * G + rb % G);
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f};
   float o[HD / 8][4];
 #pragma unroll
@@ -304,7 +334,7 @@ __global__ void __launch_bounds__(PREFILL_THREADS) attn_prefill_kernel(const Att
       cp_async_wait<0>();
     }
     __syncthreads();
-    tile_step<KT>(qf, ks, vs, tile * KT, pos_a, pos_b, p.window, score_map(p), m, l, o, lane);
+    tile_step<KT, BIAS>(qf, ks, vs, tile * KT, va, vb, p.bias_len - 1, score_map(p), m, l, o, lane);
     __syncthreads();
   }
 
@@ -354,7 +384,7 @@ static_assert(DEC_WARPS * 16 == KT, "each warp takes 16 keys of a tile");
 static_assert((DEC_WARPS * DEC_ROWS * PART_STRIDE + (DEC_WARPS + 2) * DEC_ROWS) * 4 <= 2 * DEC_STAGES * KT * LDS * 2,
               "partials and weights fit the tiles");
 
-template <int STAGES>
+template <int STAGES, bool BIAS>
 __global__ void __launch_bounds__(DEC_WARPS * 32) attn_decode_kernel(const AttnParams p) {
   extern __shared__ __align__(128) unsigned char smem[];
   __shared__ int s_last;
@@ -370,7 +400,7 @@ __global__ void __launch_bounds__(DEC_WARPS * 32) attn_decode_kernel(const AttnP
   const int row0 = p.seq_row0[b], n_new = p.seq_row0[b + 1] - row0, pos0 = p.seq_pos0[b];
   const int R = n_new * G;
   const int p_hi = pos0 + n_new - 1;
-  const int key_lo = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
+  const int key_lo = low_key(p, pos0);
   const int sp = split_pages_for(p_hi + 1);
   const int split_lo = key_lo / (sp * KT), split_hi = p_hi / (sp * KT);
   // A sequence whose new positions have no pages in its own list (or more splits than the grid
@@ -426,7 +456,8 @@ __global__ void __launch_bounds__(DEC_WARPS * 32) attn_decode_kernel(const AttnP
 #pragma unroll
     for (int i = 0; i < 4; ++i) o[j][i] = 0.0f;
   const int ra = lane >> 2, rb = ra + 8;
-  const int pos_a = ra < R ? pos0 + ra / G : -1, pos_b = rb < R ? pos0 + rb / G : -1;
+  const RowView va = row_view<BIAS>(p, ra < R ? pos0 + ra / G : -1, kvh * G + ra % G);
+  const RowView vb = row_view<BIAS>(p, rb < R ? pos0 + rb / G : -1, kvh * G + rb % G);
   uint32_t qf[HD / 16][4];
 
   for (int tile = tile_lo; tile <= tile_hi; ++tile) {
@@ -437,8 +468,8 @@ __global__ void __launch_bounds__(DEC_WARPS * 32) attn_decode_kernel(const AttnP
     if (tile == tile_lo) load_q_frags(qs, 0, lane, qf);
     // this warp's 16 keys of the tile
     const uint32_t off = (uint32_t)(warp * 16 * LDS) * 2;
-    tile_step<16>(qf, ks + off, vs + off, tile * KT + warp * 16, pos_a, pos_b, p.window, score_map(p),
-                  m, l, o, lane);
+    tile_step<16, BIAS>(qf, ks + off, vs + off, tile * KT + warp * 16, va, vb, p.bias_len - 1, score_map(p),
+                        m, l, o, lane);
     __syncthreads();                                  // the stage is free: request a later tile into it
     if (tile + STAGES <= tile_hi) {
       int pg = page_of[0];
@@ -634,6 +665,41 @@ int n_splits_for(int max_len) {
   return longs > most_short ? longs : most_short;
 }
 
+// Shared memory opt-ins of the mma.sync kernels, once per instantiation.
+template <bool BIAS>
+int configure_mma() {
+  static bool configured = false;
+  if (configured) return SB_OK;
+  cudaError_t e = cudaFuncSetAttribute(attn_prefill_kernel<BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                       PREFILL_SMEM);
+  if (e == cudaSuccess && DECODE_FITS)
+    e = cudaFuncSetAttribute(attn_decode_kernel<DEC_STAGES, BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                             DECODE_SMEM);
+  if (e == cudaSuccess && DECODE_FEW_FITS)
+    e = cudaFuncSetAttribute(attn_decode_kernel<DEC_STAGES_FEW, BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                             decode_smem(DEC_STAGES_FEW));
+  if (e == cudaSuccess && DECODE_SOME_FITS)
+    e = cudaFuncSetAttribute(attn_decode_kernel<DEC_STAGES_SOME, BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                             decode_smem(DEC_STAGES_SOME));
+  if (e != cudaSuccess)
+    SB_FAIL(SB_ERR_CUDA, "sb_attention: shared memory opt-in failed: %s", cudaGetErrorString(e));
+  configured = true;
+  return SB_OK;
+}
+
+// The decode kernel with as many stages as the grid asks for (see DEC_STAGES).
+template <bool BIAS>
+void launch_decode(const AttnParams& p, int n_sms, cudaStream_t stream) {
+  const dim3 grid(p.n_splits, p.n_kv_heads, p.n_seqs), block(DEC_WARPS * 32);
+  const long blocks = (long)p.n_splits * p.n_kv_heads * p.n_seqs;
+  if (DECODE_FEW_FITS && n_sms > 0 && blocks <= n_sms)
+    sb_launch<SB_K_ATTENTION>(attn_decode_kernel<DEC_STAGES_FEW, BIAS>, grid, block, decode_smem(DEC_STAGES_FEW), stream, p);
+  else if (DECODE_SOME_FITS && n_sms > 0 && blocks <= 2L * n_sms)
+    sb_launch<SB_K_ATTENTION>(attn_decode_kernel<DEC_STAGES_SOME, BIAS>, grid, block, decode_smem(DEC_STAGES_SOME), stream, p);
+  else
+    sb_launch<SB_K_ATTENTION>(attn_decode_kernel<DEC_STAGES, BIAS>, grid, block, DECODE_SMEM, stream, p);
+}
+
 }  // namespace
 
 #ifdef SB_ATTN_TC5
@@ -684,7 +750,7 @@ extern "C" int sb_attention(const void* q, void* out, int n_rows, int n_seqs, in
                             float scale, void* scratch, size_t scratch_bytes, int* counters,
                             int n_counters, int max_len, int n_pages, int n_sms,
                             const void* warm, size_t warm_bytes, const float* sink, float softcap,
-                            cudaStream_t stream) {
+                            int chunk, const float* bias, int bias_len, cudaStream_t stream) {
   if (hd != HD) SB_FAIL(SB_ERR_ARG, "sb_attention: built for head size %d, called with %d", HD, hd);
   if (page_size != KT)
     SB_FAIL(SB_ERR_UNSUPPORTED, "sb_attention: cache pages of %d keys (needs %d)", page_size, KT);
@@ -701,6 +767,9 @@ extern "C" int sb_attention(const void* q, void* out, int n_rows, int n_seqs, in
   AttnParams p;
   p.warm = (const char*)warm; p.warm_bytes = sb_warm_bytes(warm, warm_bytes);
   p.sink = sink;
+  if (chunk < 0 || window < 0) SB_FAIL(SB_ERR_ARG, "sb_attention: window %d, chunk %d (0: none)", window, chunk);
+  if (bias && bias_len < 1) SB_FAIL(SB_ERR_ARG, "sb_attention: a distance bias of %d entries", bias_len);
+  p.chunk = chunk; p.bias = bias; p.bias_len = bias ? bias_len : 1;
   p.q = (const bf16*)q; p.out = (bf16*)out;
   p.seq_row0 = seq_row0; p.seq_pos0 = seq_pos0; p.page_off = page_off; p.page_ids = page_ids;
   p.cache = (const bf16*)cache; p.scratch = (float*)scratch; p.counters = counters;
@@ -710,24 +779,7 @@ extern "C" int sb_attention(const void* q, void* out, int n_rows, int n_seqs, in
   p.cap_a = softcap > 0.0f ? scale / softcap : 0.0f;
   p.cap_b = softcap > 0.0f ? softcap * LOG2E : 0.0f;
   const int G = n_q_heads / n_kv_heads;
-  static bool configured = false;
-  if (!configured) {
-    cudaError_t e1 = cudaFuncSetAttribute(attn_prefill_kernel,
-                                          cudaFuncAttributeMaxDynamicSharedMemorySize, PREFILL_SMEM);
-    cudaError_t e2 = !DECODE_FITS ? cudaSuccess :
-        cudaFuncSetAttribute(attn_decode_kernel<DEC_STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                             DECODE_SMEM);
-    if (e2 == cudaSuccess && DECODE_FEW_FITS)
-      e2 = cudaFuncSetAttribute(attn_decode_kernel<DEC_STAGES_FEW>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                decode_smem(DEC_STAGES_FEW));
-    if (e2 == cudaSuccess && DECODE_SOME_FITS)
-      e2 = cudaFuncSetAttribute(attn_decode_kernel<DEC_STAGES_SOME>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                decode_smem(DEC_STAGES_SOME));
-    if (e1 != cudaSuccess || e2 != cudaSuccess)
-      SB_FAIL(SB_ERR_CUDA, "sb_attention: shared memory opt-in failed: %s",
-              cudaGetErrorString(e1 != cudaSuccess ? e1 : e2));
-    configured = true;
-  }
+  if (int rc = bias ? configure_mma<true>() : configure_mma<false>()) return rc;
   if (max_new * G <= DEC_ROWS && DECODE_FITS && n_splits_for(max_len) <= MAX_MERGE_SPLITS) {
     p.n_splits = n_splits_for(max_len);
     const size_t need = sb_attention_scratch_bytes(n_rows, n_q_heads, n_kv_heads, max_new, max_len);
@@ -760,25 +812,17 @@ extern "C" int sb_attention(const void* q, void* out, int n_rows, int n_seqs, in
     if (g_force_mma != 1 && !dt_misaligned && n_pages > 0 && n_sms > 0 && cache_rows_d < 2147483647L &&
         n_items < 2147483647L && (n_items > 10L * n_sms || g_force_mma == 2) && (size_t)(2 * p.n_splits + 3 + DT_MERGE_PARTS * HD) * sizeof(float) <= 48 * 1024 &&
         n_seqs <= 65535 && max_new * G <= 65535) {
-      static bool configured_dt = false;
-      if (!configured_dt) {
-        cudaError_t e = cudaFuncSetAttribute(attn_decode_tma_kernel,
-                                             cudaFuncAttributeMaxDynamicSharedMemorySize, DT_SMEM);
-        if (e == cudaSuccess)                          // all of the SM's memory as shared memory: three blocks fit
-          e = cudaFuncSetAttribute(attn_decode_tma_kernel, cudaFuncAttributePreferredSharedMemoryCarveout,
-                                   cudaSharedmemCarveoutMaxShared);
-        if (e != cudaSuccess)
-          SB_FAIL(SB_ERR_CUDA, "sb_attention: shared memory opt-in failed: %s", cudaGetErrorString(e));
-        configured_dt = true;
-      }
+      if (int rc = bias ? configure_decode_tma<true>() : configure_decode_tma<false>()) return rc;
       CUtensorMap map_kv;
       if (!t5_make_map(&map_kv, cache, cache_rows_d))
         SB_FAIL(SB_ERR_CUDA, "sb_attention: cuTensorMapEncodeTiled failed");
       const long slots = (long)n_sms * DT_BLOCKS_PER_SM;
       const int blocks = (int)(n_items < slots ? n_items : slots);
       if ((size_t)blocks * WARM_MAX_CHUNKS * SB_WARM_CHUNK < p.warm_bytes) p.warm_bytes = 0;
-      sb_launch<0>(attn_decode_tma_kernel, dim3(blocks), dim3(DT_THREADS), DT_SMEM, stream, map_kv, p,
-                   (int)n_items);
+      if (bias)
+        sb_launch<0>(attn_decode_tma_kernel<true>, dim3(blocks), dim3(DT_THREADS), DT_SMEM, stream, map_kv, p, (int)n_items);
+      else
+        sb_launch<0>(attn_decode_tma_kernel<false>, dim3(blocks), dim3(DT_THREADS), DT_SMEM, stream, map_kv, p, (int)n_items);
       SB_CHECK_LAUNCH("sb_attention (decode, TMA)");
       // Once: the kernel's tiles need shared memory that starts on a 1024-byte boundary, which it
       // checks itself (status 10, nothing computed).  Should that ever be reported, this step and
@@ -804,15 +848,8 @@ extern "C" int sb_attention(const void* q, void* out, int n_rows, int n_seqs, in
 #endif
     if ((size_t)p.n_splits * n_kv_heads * n_seqs * WARM_MAX_CHUNKS * SB_WARM_CHUNK < p.warm_bytes)
       p.warm_bytes = 0;
-    if (DECODE_FEW_FITS && n_sms > 0 && (long)p.n_splits * n_kv_heads * n_seqs <= n_sms)
-      sb_launch<SB_K_ATTENTION>(attn_decode_kernel<DEC_STAGES_FEW>, dim3(p.n_splits, n_kv_heads, n_seqs),
-                                dim3(DEC_WARPS * 32), decode_smem(DEC_STAGES_FEW), stream, p);
-    else if (DECODE_SOME_FITS && n_sms > 0 && (long)p.n_splits * n_kv_heads * n_seqs <= 2L * n_sms)
-      sb_launch<SB_K_ATTENTION>(attn_decode_kernel<DEC_STAGES_SOME>, dim3(p.n_splits, n_kv_heads, n_seqs),
-                                dim3(DEC_WARPS * 32), decode_smem(DEC_STAGES_SOME), stream, p);
-    else
-      sb_launch<SB_K_ATTENTION>(attn_decode_kernel<DEC_STAGES>, dim3(p.n_splits, n_kv_heads, n_seqs),
-                                dim3(DEC_WARPS * 32), DECODE_SMEM, stream, p);
+    if (bias) launch_decode<true>(p, n_sms, stream);
+    else launch_decode<false>(p, n_sms, stream);
     SB_CHECK_LAUNCH("sb_attention (decode)");
     return SB_OK;
   }
@@ -824,21 +861,15 @@ extern "C" int sb_attention(const void* q, void* out, int n_rows, int n_seqs, in
   const long cache_rows = (long)n_pages * 2 * n_kv_heads * KT;
   static bool tc5_checked = false, tc5_misaligned = false;
   if (n_pages > 0 && cache_rows < 2147483647L && scale > 0.0f && g_force_mma != 1 && !tc5_misaligned) {
-    static bool configured5 = false;
-    if (!configured5) {
-      cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc5_kernel,
-                                           cudaFuncAttributeMaxDynamicSharedMemorySize, T5_SMEM);
-      if (e != cudaSuccess)
-        SB_FAIL(SB_ERR_CUDA, "sb_attention: shared memory opt-in failed: %s", cudaGetErrorString(e));
-      configured5 = true;
-    }
+    if (int rc = bias ? configure_tc5<true>() : configure_tc5<false>()) return rc;
     CUtensorMap map_kv;
     if (!t5_make_map(&map_kv, cache, cache_rows))
       SB_FAIL(SB_ERR_CUDA, "sb_attention: cuTensorMapEncodeTiled failed");
     const long tiles5 = ((long)max_new * G + T5_QT * T5_ROWS - 1) / (T5_QT * T5_ROWS);
     if (tiles5 * n_kv_heads > 2147483647L) SB_FAIL(SB_ERR_UNSUPPORTED, "sb_attention: too many rows");
-    sb_launch<SB_K_ATTENTION>(attn_prefill_tc5_kernel, dim3((unsigned)(tiles5 * n_kv_heads), 1, n_seqs),
-              dim3(T5_THREADS), T5_SMEM, stream, map_kv, p);
+    const dim3 grid5((unsigned)(tiles5 * n_kv_heads), 1, n_seqs);
+    if (bias) sb_launch<SB_K_ATTENTION>(attn_prefill_tc5_kernel<true>, grid5, dim3(T5_THREADS), T5_SMEM, stream, map_kv, p);
+    else sb_launch<SB_K_ATTENTION>(attn_prefill_tc5_kernel<false>, grid5, dim3(T5_THREADS), T5_SMEM, stream, map_kv, p);
     SB_CHECK_LAUNCH("sb_attention (prefill, tcgen05)");
     if (tc5_checked) return SB_OK;
     // Once: the kernel's tiles need shared memory that starts on a 1024-byte boundary, which it
@@ -858,8 +889,9 @@ extern "C" int sb_attention(const void* q, void* out, int n_rows, int n_seqs, in
 #endif
   const long tiles = ((long)max_new * G + BM - 1) / BM;
   if (tiles * n_kv_heads > 2147483647L) SB_FAIL(SB_ERR_UNSUPPORTED, "sb_attention: too many rows");
-  sb_launch<SB_K_ATTENTION>(attn_prefill_kernel, dim3((unsigned)(tiles * n_kv_heads), 1, n_seqs),
-                            dim3(PREFILL_THREADS), PREFILL_SMEM, stream, p);
+  const dim3 grid((unsigned)(tiles * n_kv_heads), 1, n_seqs);
+  if (bias) sb_launch<SB_K_ATTENTION>(attn_prefill_kernel<true>, grid, dim3(PREFILL_THREADS), PREFILL_SMEM, stream, p);
+  else sb_launch<SB_K_ATTENTION>(attn_prefill_kernel<false>, grid, dim3(PREFILL_THREADS), PREFILL_SMEM, stream, p);
   SB_CHECK_LAUNCH("sb_attention (prefill)");
   return SB_OK;
 }
@@ -931,7 +963,7 @@ extern "C" int sb_attention_decode_static(const void* q, void* out, int n_rows, 
     e = cudaGetSymbolAddress(&ptr, g_static_scratch);
     if (e != cudaSuccess || !ptr)
       SB_FAIL(SB_ERR_CUDA, "%s: cudaGetSymbolAddress: %s", who, cudaGetErrorString(e));
-    e = cudaFuncSetAttribute(attn_decode_kernel<DEC_STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    e = cudaFuncSetAttribute(attn_decode_kernel<DEC_STAGES, false>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                              DECODE_SMEM);
     if (e != cudaSuccess)
       SB_FAIL(SB_ERR_CUDA, "%s: shared memory opt-in failed: %s", who, cudaGetErrorString(e));
@@ -952,9 +984,10 @@ extern "C" int sb_attention_decode_static(const void* q, void* out, int n_rows, 
   p.n_q_heads = n_q_heads; p.n_kv_heads = n_kv_heads; p.window = window; p.n_splits = n_splits;
   p.n_seqs = n_seqs;
   p.sink = nullptr;
+  p.chunk = 0; p.bias = nullptr; p.bias_len = 1;
   p.scale_log2 = scale * LOG2E;
   p.cap_a = p.cap_b = 0.0f;
-  sb_launch<SB_K_ATTENTION>(attn_decode_kernel<DEC_STAGES>, dim3(n_splits, n_kv_heads, n_seqs), dim3(DEC_WARPS * 32), DECODE_SMEM,
+  sb_launch<SB_K_ATTENTION>(attn_decode_kernel<DEC_STAGES, false>, dim3(n_splits, n_kv_heads, n_seqs), dim3(DEC_WARPS * 32), DECODE_SMEM,
             stream, p);
   SB_CHECK_LAUNCH("sb_attention_decode_static (decode)");
   return SB_OK;

@@ -6,7 +6,9 @@
 // i < j + window); s_j = (q . k_j) * scale with the scale applied after the whole dot;
 // out = sum(exp(s_j - m) v_j) / sum(exp(s_j - m)) (core/src/nn/attention.cpp:26-105,
 // 121-183).  With `sink` (one float32 per query head) the denominator also holds exp(sink_h);
-// with a cap c > 0 the score is c tanh(s_j / c).  Keys are taken in chunks whose boundaries are absolute multiples of the chunk
+// with a cap c > 0 the score is c tanh(s_j / c); with a chunk size key j is visible only from its
+// own stretch of `chunk` positions; with a distance bias [n_q_heads][bias_len] the capped score gets
+// bias[h][min(i - j, bias_len - 1)] added.  Keys are taken in chunks whose boundaries are absolute multiples of the chunk
 // length and merged in ascending order, as the reference's split decode attention does
 // (core/src/model/emit.cpp:538-544, core/src/nn/cuda_elementwise.cu:886-897), so the sum
 // depends only on the positions, not on the batch or on where the pages lie.
@@ -25,7 +27,8 @@ __global__ void __launch_bounds__(THREADS)
 attn_plain_kernel(const TQ* q, TQ* out, const int32_t* row_seq, const int32_t* row_pos,
                   const int32_t* page_off, const int32_t* page_ids, int page_size,
                   const TC* cache, int n_q_heads, int n_kv_heads,
-                  int hd, int window, float scale, const float* __restrict__ sink, float softcap) {
+                  int hd, int window, float scale, const float* __restrict__ sink, float softcap,
+                  int attn_chunk, const float* __restrict__ bias, int bias_len) {
   __shared__ float qs[MAX_HD];
   __shared__ float scores[CHUNK];
   __shared__ float bcast[3];
@@ -37,7 +40,7 @@ attn_plain_kernel(const TQ* q, TQ* out, const int32_t* row_seq, const int32_t* r
   const int pos = row_pos[t];
   const int seq = row_seq[t];
   const int32_t* pages = page_ids + page_off[seq];
-  const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+  const int lo = max(window > 0 ? max(0, pos - window + 1) : 0, attn_chunk > 0 ? max(pos, 0) / attn_chunk * attn_chunk : 0);
   // a position without a page in the sequence's own list: the row is zeros, nothing is read
   if (pos < 0 || pos / page_size >= page_off[seq + 1] - page_off[seq]) {
     for (int d = tid; d < hd; d += THREADS)
@@ -63,6 +66,7 @@ attn_plain_kernel(const TQ* q, TQ* out, const int32_t* row_seq, const int32_t* r
         for (int d = lane; d < hd; d += 32) dot = fmaf(qs[d], sb_to_f32<TC>(krow[d]), dot);
         s = sb_warp_sum(dot) * scale;
         if (softcap > 0.0f) s = softcap * tanhf(s / softcap);
+        if (bias) s += bias[(size_t)h * bias_len + min(pos - j, bias_len - 1)];
       }
       if (lane == 0) scores[j - cs] = s;
     }
@@ -138,7 +142,10 @@ extern "C" int sb_attention_plain(const void* q, void* out, int act_dtype, int n
                                   const int32_t* page_off, const int32_t* page_ids, int page_size,
                                   const void* cache, int cache_dtype, int n_q_heads,
                                   int n_kv_heads, int hd, int window, float scale,
-                                  const float* sink, float softcap, cudaStream_t stream) {
+                                  const float* sink, float softcap, int chunk, const float* bias,
+                                  int bias_len, cudaStream_t stream) {
+  if (chunk < 0 || (bias && bias_len < 1))
+    SB_FAIL(SB_ERR_ARG, "sb_attention_plain: chunk %d, a distance bias of %d entries", chunk, bias_len);
   if (softcap < 0.0f) SB_FAIL(SB_ERR_ARG, "sb_attention_plain: score cap %g (0: none)", softcap);
   if (int rc = sb_check_attention_args("sb_attention_plain", n_rows, n_q_heads, n_kv_heads, hd,
                                        window, page_size))
@@ -153,7 +160,8 @@ extern "C" int sb_attention_plain(const void* q, void* out, int act_dtype, int n
     SB_DISPATCH_DTYPE(cache_dtype, TC, {
       sb_launch(attn_plain_kernel<TQ, TC>, grid, dim3(THREADS), 0, stream,
           (const TQ*)q, (TQ*)out, row_seq, row_pos, page_off, page_ids, page_size,
-          (const TC*)cache, n_q_heads, n_kv_heads, hd, window, scale, sink, softcap);
+          (const TC*)cache, n_q_heads, n_kv_heads, hd, window, scale, sink, softcap,
+          chunk, bias, bias_len);
     });
   });
   SB_CHECK_LAUNCH("sb_attention_plain");

@@ -111,6 +111,7 @@ __device__ __forceinline__ void t5_rescale(uint32_t taddr, float factor) {
   tc_fence_before();
 }
 
+template <bool BIAS>
 __global__ void __launch_bounds__(T5_THREADS, T5_SMEM <= 115712 && T5_TMEM_COLS <= 256 ? 2 : 1)
 attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_kv, const AttnParams p) {
   extern __shared__ __align__(1024) unsigned char t5_smem[];
@@ -135,7 +136,7 @@ attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_kv, const AttnPa
   // positions without pages in the sequence's own list: nothing is read
   if (pos0 < 0 || (pos0 + n_new - 1) / KT >= p.page_off[b + 1] - p.page_off[b]) return;
   const int r_last = min(R, r_base + T5_QT * T5_ROWS) - 1;
-  const int tile_lo = (p.window > 0 ? max(0, pos0 + r_base / G - p.window + 1) : 0) / KT;
+  const int tile_lo = low_key(p, pos0 + r_base / G) / KT;
   const int tile_hi = (pos0 + r_last / G) / KT;
   const int n_tiles = tile_hi - tile_lo + 1;
   if (raw & 1023u) {                       // the swizzled tiles need this alignment
@@ -305,10 +306,12 @@ attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_kv, const AttnPa
     mbar_arrive(tb + 8 * T5_QFULL);
 
     const int r = rq_base + row;
-    const int pos = r < R ? pos0 + r / G : -1;
+    const RowView rv = row_view<BIAS>(p, r < R ? pos0 + r / G : -1, kvh * G + r % G);
+    const int bias_last = p.bias_len - 1;
     // positions of the tile's first and last real row (no real row: every page is masked)
     const int p_lo = rq_base < R ? pos0 + rq_base / G : 0x7fffffff;
     const int p_hi = rq_base < R ? pos0 + min(R - 1, rq_base + T5_ROWS - 1) / G : 0x7fffffff;
+    const int lo_hi = p_hi == 0x7fffffff ? 0 : low_key(p, p_hi);     // the last real row's first visible key
     const uint32_t o_addr = t_base + 2 * KT;
     float m_ref = -INFINITY, l = 0.0f;      // reference maximum (log2 domain) and row sum
     const ScoreMap sm = score_map(p);
@@ -329,12 +332,18 @@ attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_kv, const AttnPa
       mbar_arrive(tb + 8 * (T5_SFREE + s));
 
       // every key of the page visible to every row of the tile: no mask to apply
-      const bool open = key0 + KT - 1 <= p_lo && (p.window == 0 || p_hi - key0 < p.window);
+      const bool open = key0 + KT - 1 <= p_lo && key0 >= lo_hi;
+      if (BIAS) {
+        // a bias is not monotone in the dot product: finished scores from here on
+#pragma unroll
+        for (int i = 0; i < KT; ++i)
+          sv[i] = __float_as_uint(row_score<true>(__uint_as_float(sv[i]), sm, rv, key0 + i, bias_last));
+      }
       if (!open) {
 #pragma unroll
         for (int i = 0; i < KT; ++i) {
           const int key = key0 + i;
-          const bool seen = key <= pos && (p.window == 0 || pos - key < p.window);
+          const bool seen = key <= rv.pos && key >= rv.lo;
           if (!seen) sv[i] = __float_as_uint(-INFINITY);
         }
       }
@@ -343,7 +352,7 @@ attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_kv, const AttnPa
       for (int i = 0; i < KT; ++i) mx[i & 3] = fmaxf(mx[i & 3], __uint_as_float(sv[i]));
       // scale > 0 and the cap is monotone: the largest dot product gives the largest exponent
       const float mx_all = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));
-      const float m_tile = capped ? (mx_all == -INFINITY ? -INFINITY : mapped_score(mx_all, sm)) : mx_all * p.scale_log2;
+      const float m_tile = BIAS ? mx_all : capped ? (mx_all == -INFINITY ? -INFINITY : mapped_score(mx_all, sm)) : mx_all * p.scale_log2;
       if (__any_sync(0xffffffffu, m_tile > m_ref + T5_LAZY || (m_ref == -INFINITY && m_tile > m_ref))) {
         // move this warp's references to the rows' current maxima
         const float m_new = fmaxf(m_ref, m_tile);
@@ -361,9 +370,9 @@ attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_kv, const AttnPa
 #pragma unroll
       for (int i = 0; i < KT; i += 2) {
         const float d0 = __uint_as_float(sv[i]), d1 = __uint_as_float(sv[i + 1]);
-        const float p0 = capped ? (d0 == -INFINITY ? 0.0f : t5_ex2(mapped_score(d0, sm) - base))
+        const float p0 = BIAS ? t5_ex2(d0 - base) : capped ? (d0 == -INFINITY ? 0.0f : t5_ex2(mapped_score(d0, sm) - base))
                                 : t5_ex2(fmaf(d0, p.scale_log2, -base));
-        const float p1 = capped ? (d1 == -INFINITY ? 0.0f : t5_ex2(mapped_score(d1, sm) - base))
+        const float p1 = BIAS ? t5_ex2(d1 - base) : capped ? (d1 == -INFINITY ? 0.0f : t5_ex2(mapped_score(d1, sm) - base))
                                 : t5_ex2(fmaf(d1, p.scale_log2, -base));
         sum0 += p0;
         sum1 += p1;
@@ -418,6 +427,17 @@ inline bool t5_make_map(CUtensorMap* map, const void* cache, long rows) {
   return fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(cache), dims, strides, box,
             elem, CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B,
             CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
+}
+
+template <bool BIAS>
+int configure_tc5() {
+  static bool configured = false;
+  if (configured) return SB_OK;
+  cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc5_kernel<BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize, T5_SMEM);
+  if (e != cudaSuccess)
+    SB_FAIL(SB_ERR_CUDA, "sb_attention: shared memory opt-in failed: %s", cudaGetErrorString(e));
+  configured = true;
+  return SB_OK;
 }
 
 }  // namespace

@@ -64,6 +64,12 @@ __device__ __forceinline__ float sb_gelu_tanh(float z) {
   return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
 
+// The square of relu.
+__device__ __forceinline__ float sb_relu2(float v) {
+  const float r = fmaxf(v, 0.0f);
+  return r * r;
+}
+
 // The rotation of one pair (a at index i, b at i + rot/2): lo = a cos - b sin, hi = a sin + b cos,
 // every product and the sum rounded on its own (no fused multiply-add), so that every kernel
 // that rotates gives the same bits whatever the compiler would contract.

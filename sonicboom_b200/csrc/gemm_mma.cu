@@ -146,6 +146,8 @@ gemm_skinny_kernel(const bf16* X, const bf16* __restrict__ W, int M, int N, int 
       v += bias_dtype == SB_F32 ? load_bias<float>(bias, n) : load_bias<bf16>(bias, n);
     else if (epilogue == SB_EPI_RESIDUAL)
       v += residual[(size_t)b * N + n];
+    else if (epilogue == SB_EPI_RELU2)
+      v = sb_relu2(v);
     out[(size_t)b * N + n] = sb_from_f32<TO>(v);
   }
 }
@@ -297,6 +299,8 @@ gemm_tiled_kernel(const bf16* A, const bf16* __restrict__ W, int M, int N, int K
             v += bias_dtype == SB_F32 ? load_bias<float>(bias, n) : load_bias<bf16>(bias, n);
           else if (epilogue == SB_EPI_RESIDUAL)
             v += residual[(size_t)m * N + n];
+          else if (epilogue == SB_EPI_RELU2)
+            v = sb_relu2(v);
           out[(size_t)m * N + n] = sb_from_f32<TO>(v);
         }
       }

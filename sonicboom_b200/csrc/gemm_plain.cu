@@ -87,6 +87,8 @@ gemm_plain_kernel(const TA* A, const TW* __restrict__ W, int M, int N, int K,
                                   : __bfloat162float(((const __nv_bfloat16*)bias)[n]);
       else if (epilogue == SB_EPI_RESIDUAL)
         v += residual[(size_t)m * N + n];
+      else if (epilogue == SB_EPI_RELU2)
+        v = sb_relu2(v);
       out[(size_t)m * N + n] = sb_from_f32<TO>(v);
     }
   }
@@ -97,7 +99,7 @@ gemm_plain_kernel(const TA* A, const TW* __restrict__ W, int M, int N, int K,
 int sb_check_linear_args(const char* who, int M, int N, int K, int epilogue, const void* bias,
                          const float* residual, int out_dtype) {
   if (M <= 0 || N <= 0 || K <= 0) SB_FAIL(SB_ERR_ARG, "%s: M=%d N=%d K=%d", who, M, N, K);
-  if (epilogue < SB_EPI_NONE || epilogue > SB_EPI_SWIGLU)
+  if (epilogue < SB_EPI_NONE || epilogue > SB_EPI_RELU2)
     SB_FAIL(SB_ERR_ARG, "%s: epilogue %d", who, epilogue);
   if (epilogue == SB_EPI_BIAS && !bias) SB_FAIL(SB_ERR_ARG, "%s: bias epilogue without bias", who);
   if (epilogue == SB_EPI_RESIDUAL && !residual)

@@ -193,6 +193,9 @@ __device__ __forceinline__ void store_chunk_rowwise(const Tc5Params& p, const ui
     for (int j = 0; j < 8; ++j) {
       v[4 * j] += x[j].x; v[4 * j + 1] += x[j].y; v[4 * j + 2] += x[j].z; v[4 * j + 3] += x[j].w;
     }
+  } else if (p.epilogue == SB_EPI_RELU2) {
+#pragma unroll
+    for (int j = 0; j < 32; ++j) v[j] = sb_relu2(v[j]);
   }
   store_row((TO*)p.out + (size_t)m * p.N + n0, v, 32);
 }
@@ -243,8 +246,9 @@ __device__ __forceinline__ void store_chunk(const Tc5Params& p, float* stage, co
 #pragma unroll 8
   for (int rr = 0; rr < 32; ++rr) {
     const int m = m_base + rr;
+    const float v = stage[rr * 33 + lane] + add;
     if (m < p.M && live)
-      ((TO*)p.out)[(size_t)m * p.N + n] = sb_from_f32<TO>(stage[rr * 33 + lane] + add);
+      ((TO*)p.out)[(size_t)m * p.N + n] = sb_from_f32<TO>(p.epilogue == SB_EPI_RELU2 ? sb_relu2(v) : v);
   }
 }
 
@@ -423,6 +427,8 @@ gemm_tc5_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant
               v += p.bias_dtype == SB_F32 ? bias_at<float>(p.bias, n) : bias_at<bf16>(p.bias, n);
             else if (p.epilogue == SB_EPI_RESIDUAL)
               v += p.residual[(size_t)tok * p.N + n];
+            else if (p.epilogue == SB_EPI_RELU2)
+              v = sb_relu2(v);
             ((TO*)p.out)[(size_t)tok * p.N + n] = sb_from_f32<TO>(v);
           }
         }
@@ -618,6 +624,7 @@ tc5_reduce_kernel(const Tc5Params p, int bn) {
     else if (p.epilogue == SB_EPI_BIAS)
       v += p.bias_dtype == SB_F32 ? bias_at<float>(p.bias, o) : bias_at<bf16>(p.bias, o);
     else if (p.epilogue == SB_EPI_RESIDUAL) v += p.residual[(size_t)j * p.N + o];
+    else if (p.epilogue == SB_EPI_RELU2) v = sb_relu2(v);
     ((TO*)p.out)[(size_t)j * n_out + o] = sb_from_f32<TO>(v);
   }
 }
@@ -1065,7 +1072,7 @@ extern "C" size_t sb_gemm_tc5_scratch_bytes(int M, int N, int K, int n_sms) {
 // Whether the swapped split-K form can finish these rows with the fused reduce + norm kernel.
 static bool norm_fuses(int M, int N, int K, int n_sms, int epilogue, int out_dtype, int form) {
   const bool normal = form == 1 || (form == 0 && M > 64);
-  return !normal && M <= 64 && choose_splits(N, K, n_sms) > 1 && epilogue != SB_EPI_SWIGLU &&
+  return !normal && M <= 64 && choose_splits(N, K, n_sms) > 1 && epilogue != SB_EPI_SWIGLU && epilogue != SB_EPI_RELU2 &&
          out_dtype == SB_F32 && N % 4 == 0 && N <= RN_MAX_WIDTH;
 }
 
@@ -1110,8 +1117,8 @@ static int tc5_run(const void* A, int a_dtype, const void* W, int w_dtype, int M
   } else if (int rc = sb_check_linear_args("sb_gemm_tc5", M, N, K, epilogue, bias, residual, out_dtype))
     return rc;
   if (norm) {
-    if (epilogue == SB_EPI_SWIGLU || out_dtype != SB_F32)
-      SB_FAIL(SB_ERR_UNSUPPORTED, "sb_gemm_tc5: a norm follows a float32 product without SwiGLU");
+    if (epilogue == SB_EPI_SWIGLU || epilogue == SB_EPI_RELU2 || out_dtype != SB_F32)
+      SB_FAIL(SB_ERR_UNSUPPORTED, "sb_gemm_tc5: a norm follows a float32 product without an activation");
     if (!norm->norm_out || !sb_valid_dtype(norm->norm_weight_dtype) ||
         !sb_valid_dtype(norm->norm_out_dtype) || !(norm->norm_eps >= 0.0f))
       SB_FAIL(SB_ERR_ARG, "sb_gemm_tc5: norm output, dtype codes %d %d or eps %g",

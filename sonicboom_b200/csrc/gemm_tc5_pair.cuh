@@ -245,6 +245,9 @@ __global__ void __launch_bounds__(256) tc5_splitk_reduce_kernel(const Tc5Params 
       const float4 x = res[j];
       v[4 * j] += x.x; v[4 * j + 1] += x.y; v[4 * j + 2] += x.z; v[4 * j + 3] += x.w;
     }
+  } else if (p.epilogue == SB_EPI_RELU2) {
+#pragma unroll
+    for (int j = 0; j < 16; ++j) v[j] = sb_relu2(v[j]);
   }
   store_row((TO*)p.out + (size_t)m * p.N + n0, v, 16);
 }

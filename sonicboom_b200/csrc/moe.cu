@@ -13,6 +13,12 @@
 //   sb_moe_down:    for every tile, the expert's down product, one float32 row per pair
 //   sb_moe_combine: x[row] += sum over the row's choices, in the order of the choices, of
 //                   weight * that pair's row
+//   sb_moe_join:    the same sum where a choice may be an identity output (an id from n_experts on:
+//                   the input row itself), plus a shared expert's row that a logistic number gates, the
+//                   whole times a weight per channel; also hands the finished rows on in another dtype
+//
+// An expert is gated (gate and up matrices, the clamped activation) or plain (one up matrix, the square
+// of relu): the up products have a form for each (Up), everything else is common.
 //
 // A pair's result is a function of its own row and expert only (every output is one dot product
 // summed in a fixed order), so results do not depend on what else a step holds or on the order in
@@ -26,6 +32,10 @@ namespace {
 
 constexpr int BM = 32, BN = 64, BK = 32;      // pairs, outputs, inner values of a tile
 constexpr int GEMM_THREADS = 256;
+
+// What a tile's product does with its sums: the down product stores them per pair; the up products make
+// an activation of gate and up (GATED) or of up alone (RELU2: the square of relu).
+enum Up { DOWN = 0, GATED = 1, RELU2 = 2 };
 
 __global__ void moe_route_kernel(const float* logits, int n_rows, int n_experts, int top, int32_t* ids,
                                  float* weights) {
@@ -104,13 +114,14 @@ moe_route_warp_kernel(const float* logits, int n_rows, int n_experts, int top, i
 // choice scores, and only experts of the `keep_groups` best groups can be chosen (n_groups 1:
 // every expert can).  The `top` experts with the largest choice scores are chosen (the lower
 // index wins a tie); their weights are s_e * scale, divided by the chosen ones' sum of s when
-// `renormalize`.  All float32.  `sc` holds a warp's choice scores (minus infinity once an expert
+// `renormalize` (plus 1e-20).  With `softmax` the scores are the softmax over all experts instead.
+// A row's logits start `ld` values apart.  All float32.  `sc` holds a warp's choice scores (minus infinity once an expert
 // is chosen or its group is out), `gs` its group scores.
 constexpr int ROUTE_WARPS = 4, ROUTE_MAX_EXPERTS = 1024;
 
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
-moe_route_scored_kernel(const float* logits, const float* __restrict__ correction, int n_rows, int n_experts,
-                        int top, int n_groups, int keep_groups, int group_top, float scale, int renormalize,
+moe_route_scored_kernel(const float* logits, int ld, const float* __restrict__ correction, int n_rows, int n_experts,
+                        int softmax, int top, int n_groups, int keep_groups, int group_top, float scale, int renormalize,
                         int32_t* ids, float* weights) {
   __shared__ float sc_all[ROUTE_WARPS][ROUTE_MAX_EXPERTS];
   __shared__ float gs_all[ROUTE_WARPS][ROUTE_MAX_EXPERTS];
@@ -121,9 +132,19 @@ moe_route_scored_kernel(const float* logits, const float* __restrict__ correctio
   if (r >= n_rows) return;
   float* sc = sc_all[warp];
   float* gs = gs_all[warp];
-  const float* z = logits + (size_t)r * n_experts;
+  const float* z = logits + (size_t)r * ld;
+  float zm = 0.0f, zsum = 1.0f;                // softmax: the largest logit and the sum of exponentials
+  if (softmax) {
+    zm = -INFINITY;
+    for (int e = lane; e < n_experts; e += 32) zm = fmaxf(zm, z[e]);
+    zm = sb_warp_max(zm);
+    zsum = 0.0f;
+    for (int e = lane; e < n_experts; e += 32) zsum += expf(z[e] - zm);
+    zsum = sb_warp_sum(zsum);
+  }
+  auto score = [&](float v) { return softmax ? expf(v - zm) / zsum : 1.0f / (1.0f + expf(-v)); };
   for (int e = lane; e < n_experts; e += 32) {
-    const float s = 1.0f / (1.0f + expf(-z[e]));
+    const float s = score(z[e]);
     sc[e] = s + (correction ? correction[e] : 0.0f);
   }
   __syncwarp();
@@ -192,7 +213,7 @@ moe_route_scored_kernel(const float* logits, const float* __restrict__ correctio
         id[k] = 0;
         w[k] = 0.0f;
       } else {
-        const float s = 1.0f / (1.0f + expf(-z[best]));
+        const float s = score(z[best]);
         id[k] = best;
         w[k] = s;
         total += s;
@@ -202,9 +223,10 @@ moe_route_scored_kernel(const float* logits, const float* __restrict__ correctio
     __syncwarp();
   }
   if (lane == 0)
-    for (int k = 0; k < top; ++k) w[k] = renormalize ? w[k] / total * scale : w[k] * scale;
+    for (int k = 0; k < top; ++k) w[k] = renormalize ? w[k] / (total + 1e-20f) * scale : w[k] * scale;
 }
 
+// Pairs whose id is n_experts or more (identity outputs) have no expert and are left out.
 // meta: [0] number of tiles; then per tile (expert, first place in `order`, pairs).
 __global__ void __launch_bounds__(1024)
 moe_group_kernel(const int32_t* ids, int n_pairs, int n_experts, int tile_rows, int32_t* order, int32_t* meta) {
@@ -216,7 +238,8 @@ moe_group_kernel(const int32_t* ids, int n_pairs, int n_experts, int tile_rows, 
   for (int e = threadIdx.x; e < n_experts; e += blockDim.x) count[e] = cursor[e] = 0;
   __syncthreads();
   sb_pdl_wait();
-  for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) atomicAdd(&count[ids[p]], 1);
+  for (int p = threadIdx.x; p < n_pairs; p += blockDim.x)
+    if (ids[p] < n_experts) atomicAdd(&count[ids[p]], 1);
   __syncthreads();
   if (threadIdx.x == 0) {
     int at = 0, tiles = 0;
@@ -235,19 +258,21 @@ moe_group_kernel(const int32_t* ids, int n_pairs, int n_experts, int tile_rows, 
   __syncthreads();
   for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) {
     const int e = ids[p];
+    if (e >= n_experts) continue;
     order[start[e] + atomicAdd(&cursor[e], 1)] = p;
   }
 }
 
-// One tile of pairs of one expert times BN outputs.  GATED: a[pair's row] . (gate | up)^T with
-// the activation, written at the pair's place in `order`; else act[place] . down^T, written at the
-// pair's own index.
-template <typename TA, typename TW, bool GATED>
+// One tile of pairs of one expert times BN outputs.  An up product: a[pair's row] . (gate | up)^T (or
+// . up^T) with the activation, written at the pair's place in `order`; else act[place] . down^T, written
+// at the pair's own index.
+template <typename TA, typename TW, int UP>
 __global__ void __launch_bounds__(GEMM_THREADS)
 moe_gemm_kernel(const TA* a, const TW* __restrict__ w, const int32_t* order, const int32_t* meta, int top,
                 int n_out, int n_in, float limit, float slope, void* out_) {
+  constexpr int NW = UP == GATED ? 2 : 1;        // weight matrices of an expert
   __shared__ float As[BK][BM + 1];
-  __shared__ float Ws[GATED ? 2 : 1][BK][BN + 1];
+  __shared__ float Ws[NW][BK][BN + 1];
   __shared__ int32_t src_row[BM];
   sb_pdl_launch();
   sb_pdl_wait();
@@ -256,10 +281,10 @@ moe_gemm_kernel(const TA* a, const TW* __restrict__ w, const int32_t* order, con
   const int e = meta[1 + 3 * tile], first = meta[2 + 3 * tile], cnt = meta[3 + 3 * tile];
   const int n0 = blockIdx.y * BN;
   const int tid = threadIdx.x, tx = tid % 16, ty = tid / 16;       // 4 outputs x 2 pairs a thread
-  if (tid < BM) src_row[tid] = tid < cnt ? (GATED ? order[first + tid] / top : first + tid) : -1;
+  if (tid < BM) src_row[tid] = tid < cnt ? (UP ? order[first + tid] / top : first + tid) : -1;
   __syncthreads();
-  const TW* we = w + (size_t)e * (GATED ? 2 : 1) * n_out * n_in;
-  float acc[GATED ? 2 : 1][2][4] = {};
+  const TW* we = w + (size_t)e * NW * n_out * n_in;
+  float acc[NW][2][4] = {};
   for (int k0 = 0; k0 < n_in; k0 += BK) {
     for (int i = tid; i < BM * BK; i += GEMM_THREADS) {
       const int m = i / BK, k = i % BK;
@@ -270,14 +295,14 @@ moe_gemm_kernel(const TA* a, const TW* __restrict__ w, const int32_t* order, con
       const int n = i / BK, k = i % BK;
       const bool ok = n0 + n < n_out && k0 + k < n_in;
       Ws[0][k][n] = ok ? sb_to_f32<TW>(we[(size_t)(n0 + n) * n_in + k0 + k]) : 0.0f;
-      if (GATED) Ws[1][k][n] = ok ? sb_to_f32<TW>(we[(size_t)(n_out + n0 + n) * n_in + k0 + k]) : 0.0f;
+      if (UP == GATED) Ws[NW - 1][k][n] = ok ? sb_to_f32<TW>(we[(size_t)(n_out + n0 + n) * n_in + k0 + k]) : 0.0f;
     }
     __syncthreads();
 #pragma unroll 8
     for (int k = 0; k < BK; ++k) {
       const float a0 = As[k][ty * 2], a1 = As[k][ty * 2 + 1];
 #pragma unroll
-      for (int g = 0; g < (GATED ? 2 : 1); ++g)
+      for (int g = 0; g < NW; ++g)
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
           const float b = Ws[g][k][tx * 4 + j];
@@ -295,9 +320,10 @@ moe_gemm_kernel(const TA* a, const TW* __restrict__ w, const int32_t* order, con
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx * 4 + j;
       if (n >= n_out) continue;
-      if (GATED) {
+      if (UP) {
         TA* out = (TA*)out_;
-        out[(size_t)(first + m) * n_out + n] = sb_from_f32<TA>(sb_glu_clamped(acc[0][i][j], acc[GATED ? 1 : 0][i][j], limit, slope));
+        out[(size_t)(first + m) * n_out + n] = sb_from_f32<TA>(
+            UP == GATED ? sb_glu_clamped(acc[0][i][j], acc[NW - 1][i][j], limit, slope) : sb_relu2(acc[0][i][j]));
       } else {
         float* out = (float*)out_;
         out[(size_t)order[first + m] * n_out + n] = acc[0][i][j];
@@ -345,9 +371,9 @@ constexpr int mma_smem(int mi) { return stages_for(mi) * (mi * 32 + TN) * TK * 2
 // One tile of up to MI * 32 pairs of one expert.  2 x 4 warps, MI * 16 pairs x 32 weight rows each.
 // GATED: the 128 weight rows of a block are, for each of its four warp columns, 16 gate rows and
 // the 16 up rows of the same outputs, so a thread holds gate and up of an output side by side;
-// a block finishes 64 outputs.  Else 128 outputs of the down product.  Every output is summed over
+// a block finishes 64 outputs.  Else 128 outputs, of the plain up product or of the down product.  Every output is summed over
 // the inner values in the same order whatever the tile, the pair's place in it, or MI.
-template <int MI, bool GATED>
+template <int MI, int UP>
 __global__ void __launch_bounds__(MMA_THREADS, 2)
 moe_gemm_mma_kernel(const bf16* a, const bf16* __restrict__ w, const int32_t* order, const int32_t* meta, int top,
                     int n_out, int n_in, float limit, float slope, void* out_) {
@@ -361,12 +387,12 @@ moe_gemm_mma_kernel(const bf16* a, const bf16* __restrict__ w, const int32_t* or
   const int tile = blockIdx.x;
   if (tile >= meta[0]) return;
   const int e = meta[1 + 3 * tile], first = meta[2 + 3 * tile], cnt = meta[3 + 3 * tile];
-  const int n0 = blockIdx.y * (GATED ? TN / 2 : TN);
+  const int n0 = blockIdx.y * (UP == GATED ? TN / 2 : TN);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int warp_m = warp >> 2, warp_n = warp & 3;
-  for (int m = tid; m < TM; m += MMA_THREADS) src_row[m] = m < cnt ? (GATED ? order[first + m] / top : first + m) : -1;
+  for (int m = tid; m < TM; m += MMA_THREADS) src_row[m] = m < cnt ? (UP ? order[first + m] / top : first + m) : -1;
   __syncthreads();
-  const bf16* we = w + (size_t)e * (GATED ? 2 : 1) * n_out * n_in;
+  const bf16* we = w + (size_t)e * (UP == GATED ? 2 : 1) * n_out * n_in;
   // what this thread copies of every stage: MI chunks of the pairs' rows, 4 chunks of weight rows
   const int chunk = tid & 7;
   const bf16* a_src[MI];
@@ -380,7 +406,7 @@ moe_gemm_mma_kernel(const bf16* a, const bf16* __restrict__ w, const int32_t* or
   for (int i = 0; i < 4; ++i) {
     const int rr = (tid >> 3) + i * 32;
     int n;
-    if (GATED) {
+    if (UP == GATED) {
       n = n0 + (rr >> 5) * 16 + (rr & 15);
       n = n < n_out ? ((rr & 16) ? n_out + n : n) : -1;
     } else {
@@ -454,7 +480,7 @@ moe_gemm_mma_kernel(const bf16* a, const bf16* __restrict__ w, const int32_t* or
     for (int half = 0; half < 2; ++half) {
       const int m = warp_m * (MI * 16) + i * 16 + g + half * 8;
       if (m >= cnt) continue;
-      if (GATED) {
+      if (UP == GATED) {
         bf16* out = (bf16*)out_ + (size_t)(first + m) * n_out;
 #pragma unroll
         for (int j = 0; j < 2; ++j)
@@ -464,6 +490,16 @@ moe_gemm_mma_kernel(const bf16* a, const bf16* __restrict__ w, const int32_t* or
             if (n < n_out)
               out[n] = __float2bfloat16(sb_glu_clamped(acc[i][j][half * 2 + c], acc[i][j + 2][half * 2 + c], limit, slope));
           }
+      } else if (UP == RELU2) {
+        // columns 2t and 2t + 1 as one 4-byte store (n_out is a multiple of 8 here)
+        bf16* out = (bf16*)out_ + (size_t)(first + m) * n_out;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const int n = n0 + warp_n * 32 + j * 8 + 2 * t;
+          if (n < n_out)
+            *reinterpret_cast<__nv_bfloat162*>(out + n) =
+                __floats2bfloat162_rn(sb_relu2(acc[i][j][half * 2]), sb_relu2(acc[i][j][half * 2 + 1]));
+        }
       } else {
         float* out = (float*)out_ + (size_t)order[first + m] * n_out;
 #pragma unroll
@@ -478,18 +514,19 @@ moe_gemm_mma_kernel(const bf16* a, const bf16* __restrict__ w, const int32_t* or
   }
 }
 
-template <int MI, bool GATED>
+template <int MI, int UP>
 int launch_mma(const void* a, const void* w, const int32_t* order, const int32_t* meta, int tiles, int top, int n_out,
                int n_in, float limit, float slope, void* out, cudaStream_t stream) {
   static bool opted = false;
   if (!opted) {
-    cudaError_t e = cudaFuncSetAttribute(moe_gemm_mma_kernel<MI, GATED>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    cudaError_t e = cudaFuncSetAttribute(moe_gemm_mma_kernel<MI, UP>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          mma_smem(MI));
     if (e != cudaSuccess) SB_FAIL(SB_ERR_CUDA, "mixture of experts: shared memory opt-in failed: %s", cudaGetErrorString(e));
     opted = true;
   }
-  const dim3 grid(tiles, (n_out + (GATED ? TN / 2 : TN) - 1) / (GATED ? TN / 2 : TN));
-  sb_launch<SB_K_OTHER>(moe_gemm_mma_kernel<MI, GATED>, grid, dim3(MMA_THREADS), (size_t)mma_smem(MI), stream,
+  constexpr int per = UP == GATED ? TN / 2 : TN;
+  const dim3 grid(tiles, (n_out + per - 1) / per);
+  sb_launch<SB_K_OTHER>(moe_gemm_mma_kernel<MI, UP>, grid, dim3(MMA_THREADS), (size_t)mma_smem(MI), stream,
                         (const bf16*)a, (const bf16*)w, order, meta, top, n_out, n_in, limit, slope, out);
   return SB_OK;
 }
@@ -502,6 +539,85 @@ __global__ void moe_combine_kernel(float* x, const float* pair_out, const float*
     float s = 0.0f;
     for (int k = 0; k < top; ++k) s = fmaf(weights[r * top + k], pair_out[(r * top + k) * width + c], s);
     x[r * width + c] += s;
+  }
+}
+
+// y = sum over the row's choices, in their order, of weight * (the pair's row, or the input row h for an
+// identity output), + sigmoid(gate) * the shared expert's row; x += scale * y; copy = x.
+template <int V>
+struct Lanes {
+  float v[V];
+};
+template <int V, typename T>
+__device__ __forceinline__ Lanes<V> load_lanes(const T* p) {
+  Lanes<V> r;
+  if constexpr (V == 4 && sizeof(T) == 4) {
+    const float4 f = *reinterpret_cast<const float4*>(p);
+    r.v[0] = f.x; r.v[1] = f.y; r.v[2] = f.z; r.v[3] = f.w;
+  } else if constexpr (V == 4) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+    r.v[0] = a.x; r.v[1] = a.y; r.v[2] = b.x; r.v[3] = b.y;
+  } else {
+#pragma unroll
+    for (int i = 0; i < V; ++i) r.v[i] = sb_to_f32<T>(p[i]);
+  }
+  return r;
+}
+
+template <int V, typename TH, typename TS, typename TC>
+__global__ void __launch_bounds__(256)
+moe_join_kernel(float* x, const float* pair_out, const int32_t* ids, const float* weights, int n_experts,
+                const TH* h, const float* shared, const float* gate, int gate_ld, const TS* __restrict__ scale,
+                int top, int width, TC* copy) {
+  sb_pdl_launch();
+  sb_pdl_wait();
+  const size_t r = blockIdx.x;
+  const float g = gate ? 1.0f / (1.0f + expf(-gate[r * gate_ld])) : 1.0f;
+  for (int c = (blockIdx.y * blockDim.x + threadIdx.x) * V; c < width; c += gridDim.y * blockDim.x * V) {
+    Lanes<V> s;
+#pragma unroll
+    for (int i = 0; i < V; ++i) s.v[i] = 0.0f;
+    const Lanes<V> own = load_lanes<V>(h + r * width + c);
+#pragma unroll 4
+    for (int k = 0; k < top; ++k) {
+      const float wk = weights[r * top + k];
+      const Lanes<V> y = ids[r * top + k] < n_experts ? load_lanes<V>(pair_out + (r * top + k) * width + c) : own;
+#pragma unroll
+      for (int i = 0; i < V; ++i) s.v[i] = fmaf(wk, y.v[i], s.v[i]);
+    }
+    if (shared) {
+      const Lanes<V> y = load_lanes<V>(shared + r * width + c);
+#pragma unroll
+      for (int i = 0; i < V; ++i) s.v[i] = fmaf(g, y.v[i], s.v[i]);
+    }
+    Lanes<V> o = load_lanes<V>(x + r * width + c);
+    if (scale) {
+      const Lanes<V> w = load_lanes<V>(scale + c);
+#pragma unroll
+      for (int i = 0; i < V; ++i) o.v[i] += w.v[i] * s.v[i];
+    } else {
+#pragma unroll
+      for (int i = 0; i < V; ++i) o.v[i] += s.v[i];
+    }
+    if constexpr (V == 4) {
+      *reinterpret_cast<float4*>(x + r * width + c) = make_float4(o.v[0], o.v[1], o.v[2], o.v[3]);
+    } else {
+      x[r * width + c] = o.v[0];
+    }
+    if (copy) {
+      if constexpr (V == 4 && sizeof(TC) == 2) {
+        __nv_bfloat162 a = __floats2bfloat162_rn(o.v[0], o.v[1]), b = __floats2bfloat162_rn(o.v[2], o.v[3]);
+        uint2 u;
+        u.x = *reinterpret_cast<uint32_t*>(&a);
+        u.y = *reinterpret_cast<uint32_t*>(&b);
+        *reinterpret_cast<uint2*>(copy + r * width + c) = u;
+      } else {
+#pragma unroll
+        for (int i = 0; i < V; ++i) copy[r * width + c + i] = sb_from_f32<TC>(o.v[i]);
+      }
+    }
   }
 }
 
@@ -521,11 +637,12 @@ extern "C" int sb_moe_route(const float* logits, int n_rows, int n_experts, int 
   return SB_OK;
 }
 
-extern "C" int sb_moe_route_scored(const float* logits, const float* correction, int n_rows, int n_experts, int top,
-                                   int n_groups, int keep_groups, int group_top, float scale, int renormalize,
+extern "C" int sb_moe_route_scored(const float* logits, int ld, const float* correction, int n_rows, int n_experts,
+                                   int softmax, int top, int n_groups, int keep_groups, int group_top, float scale, int renormalize,
                                    int32_t* ids, float* weights, cudaStream_t stream) {
   if (n_rows <= 0 || n_experts <= 0 || top <= 0 || top > n_experts || !logits || !ids || !weights)
     SB_FAIL(SB_ERR_ARG, "sb_moe_route_scored: rows=%d experts=%d top=%d", n_rows, n_experts, top);
+  if (ld < n_experts) SB_FAIL(SB_ERR_ARG, "sb_moe_route_scored: rows of %d logits for %d experts", ld, n_experts);
   if (n_experts > ROUTE_MAX_EXPERTS)
     SB_FAIL(SB_ERR_UNSUPPORTED, "sb_moe_route_scored: %d experts (at most %d)", n_experts, ROUTE_MAX_EXPERTS);
   if (n_groups < 1 || n_experts % n_groups || keep_groups < 1 || keep_groups > n_groups || group_top < 1)
@@ -535,7 +652,7 @@ extern "C" int sb_moe_route_scored(const float* logits, const float* correction,
     SB_FAIL(SB_ERR_ARG, "sb_moe_route_scored: %d kept groups of %d experts cannot give %d choices", keep_groups,
             n_experts / n_groups, top);
   sb_launch<SB_K_ELEMENTWISE>(moe_route_scored_kernel, dim3((n_rows + ROUTE_WARPS - 1) / ROUTE_WARPS),
-                              dim3(ROUTE_WARPS * 32), 0, stream, logits, correction, n_rows, n_experts, top, n_groups,
+                              dim3(ROUTE_WARPS * 32), 0, stream, logits, ld, correction, n_rows, n_experts, softmax, top, n_groups,
                               keep_groups, group_top, scale, renormalize, ids, weights);
   SB_CHECK_LAUNCH("sb_moe_route_scored");
   return SB_OK;
@@ -566,7 +683,9 @@ extern "C" int sb_moe_group(const int32_t* ids, int n_pairs, int n_experts, int 
 
 extern "C" int sb_moe_up(const void* a, int a_dtype, const void* w, int w_dtype, const int32_t* order,
                          const int32_t* meta, int n_pairs, int n_experts, int tile_rows, int top, int ff, int width,
-                         float limit, float slope, void* act, cudaStream_t stream) {
+                         int kind, float limit, float slope, void* act, cudaStream_t stream) {
+  if (kind != SB_EXPERT_CLAMPED && kind != SB_EXPERT_RELU2) SB_FAIL(SB_ERR_ARG, "sb_moe_up: expert kind %d", kind);
+  const bool gated = kind == SB_EXPERT_CLAMPED;
   if (n_pairs <= 0 || n_experts <= 0 || top <= 0 || ff <= 0 || width <= 0 || !a || !w || !order || !meta || !act)
     SB_FAIL(SB_ERR_ARG, "sb_moe_up: pairs=%d experts=%d top=%d ff=%d width=%d", n_pairs, n_experts, top, ff, width);
   if (!sb_valid_dtype(a_dtype) || a_dtype != w_dtype) SB_FAIL(SB_ERR_ARG, "sb_moe_up: dtype codes %d %d", a_dtype, w_dtype);
@@ -575,16 +694,22 @@ extern "C" int sb_moe_up(const void* a, int a_dtype, const void* w, int w_dtype,
   const int tiles = sb_moe_max_tiles(n_pairs, n_experts, tile_rows);
   if (tile_rows != BM) {
     if (((uintptr_t)a | (uintptr_t)w) & 15) SB_FAIL(SB_ERR_ARG, "sb_moe_up: operands must be 16-byte aligned");
-    const int rc = tile_rows == 128 ? launch_mma<4, true>(a, w, order, meta, tiles, top, ff, width, limit, slope, act, stream)
-                                    : launch_mma<2, true>(a, w, order, meta, tiles, top, ff, width, limit, slope, act, stream);
+#define SB_MOE_UP(MI) (gated ? launch_mma<MI, GATED>(a, w, order, meta, tiles, top, ff, width, limit, slope, act, stream) \
+                             : launch_mma<MI, RELU2>(a, w, order, meta, tiles, top, ff, width, limit, slope, act, stream))
+    const int rc = tile_rows == 128 ? SB_MOE_UP(4) : SB_MOE_UP(2);
+#undef SB_MOE_UP
     if (rc) return rc;
     SB_CHECK_LAUNCH("sb_moe_up");
     return SB_OK;
   }
   const dim3 grid(tiles, (ff + BN - 1) / BN);
   SB_DISPATCH_DTYPE(a_dtype, T, {
-    sb_launch<SB_K_OTHER>(moe_gemm_kernel<T, T, true>, grid, dim3(GEMM_THREADS), 0, stream, (const T*)a, (const T*)w, order,
-                          meta, top, ff, width, limit, slope, act);
+    if (gated)
+      sb_launch<SB_K_OTHER>(moe_gemm_kernel<T, T, GATED>, grid, dim3(GEMM_THREADS), 0, stream, (const T*)a, (const T*)w,
+                            order, meta, top, ff, width, limit, slope, act);
+    else
+      sb_launch<SB_K_OTHER>(moe_gemm_kernel<T, T, RELU2>, grid, dim3(GEMM_THREADS), 0, stream, (const T*)a, (const T*)w,
+                            order, meta, top, ff, width, limit, slope, act);
   });
   SB_CHECK_LAUNCH("sb_moe_up");
   return SB_OK;
@@ -602,15 +727,15 @@ extern "C" int sb_moe_down(const void* act, int a_dtype, const void* w, int w_dt
   if (tile_rows != BM) {
     if (((uintptr_t)act | (uintptr_t)w) & 15) SB_FAIL(SB_ERR_ARG, "sb_moe_down: operands must be 16-byte aligned");
     const int rc = tile_rows == 128
-                       ? launch_mma<4, false>(act, w, order, meta, tiles, top, width, ff, 0.0f, 0.0f, pair_out, stream)
-                       : launch_mma<2, false>(act, w, order, meta, tiles, top, width, ff, 0.0f, 0.0f, pair_out, stream);
+                       ? launch_mma<4, DOWN>(act, w, order, meta, tiles, top, width, ff, 0.0f, 0.0f, pair_out, stream)
+                       : launch_mma<2, DOWN>(act, w, order, meta, tiles, top, width, ff, 0.0f, 0.0f, pair_out, stream);
     if (rc) return rc;
     SB_CHECK_LAUNCH("sb_moe_down");
     return SB_OK;
   }
   const dim3 grid(tiles, (width + BN - 1) / BN);
   SB_DISPATCH_DTYPE(a_dtype, T, {
-    sb_launch<SB_K_OTHER>(moe_gemm_kernel<T, T, false>, grid, dim3(GEMM_THREADS), 0, stream, (const T*)act, (const T*)w, order,
+    sb_launch<SB_K_OTHER>(moe_gemm_kernel<T, T, DOWN>, grid, dim3(GEMM_THREADS), 0, stream, (const T*)act, (const T*)w, order,
                           meta, top, width, ff, 0.0f, 0.0f, (void*)pair_out);
   });
   SB_CHECK_LAUNCH("sb_moe_down");
@@ -625,5 +750,34 @@ extern "C" int sb_moe_combine(float* x, const float* pair_out, const float* weig
   sb_launch<SB_K_ELEMENTWISE>(moe_combine_kernel, dim3(n_rows, by < 64 ? by : 64), dim3(256), 0, stream, x, pair_out, weights,
                               top, width);
   SB_CHECK_LAUNCH("sb_moe_combine");
+  return SB_OK;
+}
+
+extern "C" int sb_moe_join(float* x, const float* pair_out, const int32_t* ids, const float* weights, int n_experts,
+                           const void* h, int h_dtype, const float* shared, const float* gate, int gate_ld,
+                           const void* scale, int scale_dtype, int n_rows, int top, int width, void* copy,
+                           int copy_dtype, cudaStream_t stream) {
+  if (n_rows <= 0 || top <= 0 || width <= 0 || n_experts <= 0 || !x || !pair_out || !ids || !weights || !h)
+    SB_FAIL(SB_ERR_ARG, "sb_moe_join: rows=%d top=%d width=%d experts=%d", n_rows, top, width, n_experts);
+  if (!sb_valid_dtype(h_dtype) || (scale && !sb_valid_dtype(scale_dtype)) || (copy && !sb_valid_dtype(copy_dtype)))
+    SB_FAIL(SB_ERR_ARG, "sb_moe_join: dtype codes %d %d %d", h_dtype, scale_dtype, copy_dtype);
+  if (gate && !shared) SB_FAIL(SB_ERR_ARG, "sb_moe_join: a gate without a shared expert's rows");
+  const bool vec = width % 4 == 0 && (((uintptr_t)x | (uintptr_t)pair_out | (uintptr_t)shared | (uintptr_t)h |
+                                       (uintptr_t)scale | (uintptr_t)copy) & 15) == 0;
+  const int per = 256 * (vec ? 4 : 1), chunks = (width + per - 1) / per;
+  const dim3 grid(n_rows, n_rows >= 2048 ? 1 : (chunks < 64 ? chunks : 64));
+  SB_DISPATCH_DTYPE(h_dtype, TH, {
+    SB_DISPATCH_DTYPE(scale ? scale_dtype : SB_F32, TS, {
+      SB_DISPATCH_DTYPE(copy ? copy_dtype : SB_F32, TC, {
+        if (vec)
+          sb_launch<SB_K_ELEMENTWISE>(moe_join_kernel<4, TH, TS, TC>, grid, dim3(256), 0, stream, x, pair_out, ids, weights,
+                                      n_experts, (const TH*)h, shared, gate, gate_ld, (const TS*)scale, top, width, (TC*)copy);
+        else
+          sb_launch<SB_K_ELEMENTWISE>(moe_join_kernel<1, TH, TS, TC>, grid, dim3(256), 0, stream, x, pair_out, ids, weights,
+                                      n_experts, (const TH*)h, shared, gate, gate_ld, (const TS*)scale, top, width, (TC*)copy);
+      });
+    });
+  });
+  SB_CHECK_LAUNCH("sb_moe_join");
   return SB_OK;
 }

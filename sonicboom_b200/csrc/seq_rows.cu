@@ -4,10 +4,11 @@
 //                       previous and the current token (the previous token of a step's first
 //                       row comes from per-slot state)
 //   sb_keep_last_token: a step's last token of every sequence into that state
-//   sb_layernorm:       (x - mean) / sqrt(var + eps) * w, no bias
+//   sb_layernorm:       (x - mean) / sqrt(var + eps) * w [+ b]
 //   sb_causal_conv:     a short causal convolution over time on every channel, reading the
 //                       taps before a step's first row from per-slot state
-//   sb_conv_state:      a step's last taps - 1 inputs of every sequence into that state
+//   sb_conv_heads:      the same convolution over a fused q|k|v projection, its results going straight to
+//                       the query rows and the cache pages
 //
 // All arithmetic is float32; sums over a row are fixed trees.
 #include <math.h>
@@ -69,7 +70,8 @@ __global__ void keep_last_token_kernel(const int32_t* tokens, const int32_t* seq
 
 template <int NT, typename TW, typename TO>
 __global__ void __launch_bounds__(NT)
-layernorm_kernel(const float* x, const int32_t* rows, int width, const TW* __restrict__ w, float eps, TO* out) {
+layernorm_kernel(const float* x, const int32_t* rows, int width, const TW* __restrict__ w,
+                 const TW* __restrict__ b, float eps, TO* out) {
   __shared__ float red[NT / 32 + 1];
   sb_pdl_launch();
   sb_pdl_wait();
@@ -85,8 +87,10 @@ layernorm_kernel(const float* x, const int32_t* rows, int width, const TW* __res
   }
   const float inv = 1.0f / sqrtf(block_sum<NT>(q, red) / (float)width + eps);
   TO* o = out + (size_t)blockIdx.x * width;
-  for (int i = threadIdx.x; i < width; i += NT)
-    o[i] = sb_from_f32<TO>(((xr[i] - mean) * inv) * sb_to_f32<TW>(w[i]));
+  for (int i = threadIdx.x; i < width; i += NT) {
+    const float v = ((xr[i] - mean) * inv) * sb_to_f32<TW>(w[i]);
+    o[i] = sb_from_f32<TO>(b ? v + sb_to_f32<TW>(b[i]) : v);
+  }
 }
 
 // y_t = [x_t +] [bias +] sum_j w[c, j] x_(t - taps + 1 + j), optionally through silu.  A tap before
@@ -128,6 +132,7 @@ __global__ void causal_conv_kernel(const float* x, int ld, int x_off, int channe
 // CONV_RUN consecutive rows of its channel and keeps the last taps - 1 inputs in registers, so a row
 // is read once instead of once per tap.  Every sum has the order of the kernel above.
 constexpr int CONV_MAXT = 8, CONV_RUN = 8;
+constexpr int CONV_HEADS_TAPS = 5;      // most taps of sb_conv_heads
 template <typename TW, typename TO>
 __global__ void causal_conv_run_kernel(const float* x, int n_rows, int ld, int x_off, int channels, int taps,
                                        const TW* __restrict__ w, const TW* __restrict__ bias, int act, int add_input,
@@ -167,6 +172,147 @@ __global__ void causal_conv_run_kernel(const float* x, int n_rows, int ld, int x
 #pragma unroll
     for (int d = CONV_MAXT - 1; d >= 1; --d) hist[d] = hist[d - 1];
   }
+}
+
+// The convolution of a fused projection row [q heads x dim | k heads x dim | v heads x vdim] whose
+// results are attention's operands: query channels go to q_out [row][head][hd], key and value channels
+// to the position's cache row (key plane, value plane), both padded with zeros to hd.  A thread takes V
+// neighbouring channels of one head and CONV_RUN consecutive rows (one row with OWN: every sequence
+// brings one, and the thread shifts its channels' state).  The sums are those of the kernels above.
+struct HeadsArgs {
+  const float* proj;
+  int n_rows, ld;
+  int hq, hkv, dim, vdim, hd;          // channels: hq * dim, hkv * dim, hkv * vdim
+  const void* w;                       // [channels, taps]
+  const int32_t* row_seq;
+  const int32_t* row_pos;
+  const int32_t* seq_pos0;
+  const int32_t* seq_slot;
+  const int32_t* page_off;
+  const int32_t* page_ids;
+  int page_size;
+  float* state;                        // [slot, taps - 1, channels] or null (one tap)
+  void* cache;
+  void* q_out;
+};
+
+template <int V, typename T>
+__device__ __forceinline__ void put_lanes(T* p, const float (&v)[V]) {
+  if constexpr (V == 4 && sizeof(T) == 2) {
+    __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
+    uint2 u;
+    u.x = *reinterpret_cast<uint32_t*>(&a);
+    u.y = *reinterpret_cast<uint32_t*>(&b);
+    *reinterpret_cast<uint2*>(p) = u;
+  } else if constexpr (V == 4) {
+    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+  } else {
+    p[0] = sb_from_f32<T>(v[0]);
+  }
+}
+template <int V>
+__device__ __forceinline__ void get_lanes(const float* p, float (&v)[V]) {
+  if constexpr (V == 4) {
+    const float4 f = *reinterpret_cast<const float4*>(p);
+    v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+  } else {
+    v[0] = p[0];
+  }
+}
+
+template <int TAPS, int V, typename TW, typename T, bool OWN>
+__global__ void __launch_bounds__(128) conv_heads_kernel(const HeadsArgs p) {
+  sb_pdl_launch();
+  const int qw = p.hq * p.dim, kw = p.hkv * p.dim, vw = p.hkv * p.vdim, channels = qw + kw + vw;
+  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
+  if (c >= channels) return;
+  const int part = c < qw ? 0 : (c < qw + kw ? 1 : 2);
+  const int local = part == 0 ? c : (part == 1 ? c - qw : c - qw - kw);
+  const int size = part == 2 ? p.vdim : p.dim, head = local / size, d = local % size;
+  float wd[TAPS][V];                   // by distance: the weight of the input `i` rows before
+#pragma unroll
+  for (int i = 0; i < TAPS; ++i)
+#pragma unroll
+    for (int j = 0; j < V; ++j) wd[i][j] = sb_to_f32<TW>(((const TW*)p.w)[(size_t)(c + j) * TAPS + (TAPS - 1 - i)]);
+  sb_pdl_wait();
+  const int r_begin = blockIdx.x * (OWN ? 1 : CONV_RUN), r_end = OWN ? r_begin + 1 : min(p.n_rows, r_begin + CONV_RUN);
+  float hist[TAPS][V];
+  if (!OWN) {
+#pragma unroll
+    for (int i = 1; i < TAPS; ++i) {
+      if (r_begin - i >= 0) {
+        get_lanes<V>(p.proj + (size_t)(r_begin - i) * p.ld + c, hist[i]);
+      } else {
+#pragma unroll
+        for (int j = 0; j < V; ++j) hist[i][j] = 0.0f;
+      }
+    }
+  }
+  for (int r = r_begin; r < r_end; ++r) {
+    const int s = p.row_seq[r], pos = p.row_pos[r], pos0 = OWN ? pos : p.seq_pos0[s];
+    float* st = p.state ? p.state + (size_t)p.seq_slot[s] * (TAPS - 1) * channels + c : nullptr;
+    get_lanes<V>(p.proj + (size_t)r * p.ld + c, hist[0]);
+    float acc[V];
+#pragma unroll
+    for (int j = 0; j < V; ++j) acc[j] = 0.0f;
+#pragma unroll
+    for (int i = TAPS - 1; i >= 0; --i) {
+      const int at = pos - i;                      // before the step's first row: the state; before the start: zero
+      float v[V];
+      if (at >= pos0) {
+#pragma unroll
+        for (int j = 0; j < V; ++j) v[j] = hist[i][j];
+      } else if (at >= 0) {
+        get_lanes<V>(st + (size_t)(at - pos0 + TAPS - 1) * channels, v);
+        if (OWN)
+#pragma unroll
+          for (int j = 0; j < V; ++j) hist[i][j] = v[j];
+      } else {
+#pragma unroll
+        for (int j = 0; j < V; ++j) {
+          v[j] = 0.0f;
+          if (OWN) hist[i][j] = 0.0f;
+        }
+      }
+#pragma unroll
+      for (int j = 0; j < V; ++j) acc[j] = fmaf(wd[i][j], v[j], acc[j]);
+    }
+    T* dst = nullptr;
+    if (part == 0) {
+      dst = (T*)p.q_out + ((size_t)r * p.hq + head) * p.hd;
+    } else {
+      const int first = p.page_off[s], pi = pos / p.page_size;
+      const int page = pos >= 0 && pi < p.page_off[s + 1] - first ? p.page_ids[first + pi] : -1;
+      if (page >= 0)                               // else no page of its own there: nothing is written
+        dst = (T*)p.cache + ((((size_t)page * 2 + (part == 2)) * p.hkv + head) * p.page_size + pos % p.page_size) * p.hd;
+    }
+    if (dst) {
+      put_lanes<V>(dst + d, acc);
+      if (d == 0)
+        for (int e = size; e < p.hd; ++e) dst[e] = sb_from_f32<T>(0.0f);
+    }
+    if (OWN) {
+      if (TAPS > 1 && st) {
+#pragma unroll
+        for (int i = 0; i + 1 < TAPS; ++i) put_lanes<V>(st + (size_t)i * channels, hist[TAPS - 2 - i]);   // place i: input TAPS - 2 - i rows back
+      }
+    } else {
+#pragma unroll
+      for (int i = TAPS - 1; i >= 1; --i)
+#pragma unroll
+        for (int j = 0; j < V; ++j) hist[i][j] = hist[i - 1][j];
+    }
+  }
+}
+
+template <int TAPS, typename TW, typename T>
+void launch_conv_heads(const HeadsArgs& a, bool own, bool vec, cudaStream_t stream) {
+  const int channels = a.hq * a.dim + a.hkv * (a.dim + a.vdim), per = 128 * (vec ? 4 : 1);
+  const dim3 grid(own ? a.n_rows : (a.n_rows + CONV_RUN - 1) / CONV_RUN, (channels + per - 1) / per);
+  if (own && vec) sb_launch<SB_K_ELEMENTWISE>(conv_heads_kernel<TAPS, 4, TW, T, true>, grid, dim3(128), 0, stream, a);
+  else if (own) sb_launch<SB_K_ELEMENTWISE>(conv_heads_kernel<TAPS, 1, TW, T, true>, grid, dim3(128), 0, stream, a);
+  else if (vec) sb_launch<SB_K_ELEMENTWISE>(conv_heads_kernel<TAPS, 4, TW, T, false>, grid, dim3(128), 0, stream, a);
+  else sb_launch<SB_K_ELEMENTWISE>(conv_heads_kernel<TAPS, 1, TW, T, false>, grid, dim3(128), 0, stream, a);
 }
 
 __global__ void conv_state_kernel(const float* x, int ld, int x_off, int channels, int taps,
@@ -213,7 +359,7 @@ extern "C" int sb_keep_last_token(const int32_t* tokens, const int32_t* seq_row0
 }
 
 extern "C" int sb_layernorm(const float* x, const int32_t* rows, int n_rows, int width, const void* weight,
-                            int weight_dtype, float eps, void* out, int out_dtype, cudaStream_t stream) {
+                            const void* bias, int weight_dtype, float eps, void* out, int out_dtype, cudaStream_t stream) {
   if (n_rows <= 0 || width <= 0 || !x || !weight || !out) SB_FAIL(SB_ERR_ARG, "sb_layernorm: rows=%d width=%d", n_rows, width);
   if (!sb_valid_dtype(weight_dtype) || !sb_valid_dtype(out_dtype))
     SB_FAIL(SB_ERR_ARG, "sb_layernorm: dtype codes %d %d", weight_dtype, out_dtype);
@@ -221,10 +367,10 @@ extern "C" int sb_layernorm(const float* x, const int32_t* rows, int n_rows, int
     SB_DISPATCH_DTYPE(out_dtype, TO, {
       if (n_rows >= 512 || width <= 1024)
         sb_launch<SB_K_ELEMENTWISE>(layernorm_kernel<256, TW, TO>, dim3(n_rows), dim3(256), 0, stream, x, rows, width,
-                                    (const TW*)weight, eps, (TO*)out);
+                                    (const TW*)weight, (const TW*)bias, eps, (TO*)out);
       else
         sb_launch<SB_K_ELEMENTWISE>(layernorm_kernel<1024, TW, TO>, dim3(n_rows), dim3(1024), 0, stream, x, rows, width,
-                                    (const TW*)weight, eps, (TO*)out);
+                                    (const TW*)weight, (const TW*)bias, eps, (TO*)out);
     });
   });
   SB_CHECK_LAUNCH("sb_layernorm");
@@ -268,6 +414,51 @@ extern "C" int sb_causal_conv(const float* x, int n_rows, int ld, int x_off, int
     sb_launch<SB_K_ELEMENTWISE>(conv_state_kernel, dim3(n_seqs, (channels + nt - 1) / nt), dim3(nt), 0, stream, x, ld,
                                 x_off, channels, taps, seq_row0, seq_slot, state);
     SB_CHECK_LAUNCH("sb_causal_conv (state)");
+  }
+  return SB_OK;
+}
+
+extern "C" int sb_conv_heads_max_taps(void) { return CONV_HEADS_TAPS; }
+
+extern "C" int sb_conv_heads(const float* proj, int n_rows, int ld, int n_q_heads, int n_kv_heads, int dim, int vdim,
+                             int hd, int taps, const void* w, int w_dtype, int n_seqs, const int32_t* row_seq,
+                             const int32_t* row_pos, const int32_t* seq_row0, const int32_t* seq_pos0,
+                             const int32_t* seq_slot, const int32_t* page_off, const int32_t* page_ids,
+                             int page_size, float* state, void* cache, void* q_out, int dtype, cudaStream_t stream) {
+  if (n_rows <= 0 || n_seqs <= 0 || n_q_heads <= 0 || n_kv_heads <= 0 || dim <= 0 || vdim <= 0 || hd < dim || hd < vdim)
+    SB_FAIL(SB_ERR_ARG, "sb_conv_heads: rows=%d seqs=%d heads=%d/%d dim=%d vdim=%d hd=%d", n_rows, n_seqs, n_q_heads,
+            n_kv_heads, dim, vdim, hd);
+  if (taps < 1 || taps > CONV_HEADS_TAPS)
+    SB_FAIL(SB_ERR_UNSUPPORTED, "sb_conv_heads: %d taps (1 to %d)", taps, CONV_HEADS_TAPS);
+  if (!proj || !w || !row_seq || !row_pos || !seq_row0 || !seq_pos0 || !seq_slot || !page_off || !page_ids || page_size <= 0 ||
+      (taps > 1 && !state) || !cache || !q_out)
+    SB_FAIL(SB_ERR_ARG, "sb_conv_heads: arguments missing");
+  if (!sb_valid_dtype(w_dtype) || !sb_valid_dtype(dtype)) SB_FAIL(SB_ERR_ARG, "sb_conv_heads: dtype codes %d %d", w_dtype, dtype);
+  const int channels = n_q_heads * dim + n_kv_heads * (dim + vdim);
+  if (channels > ld) SB_FAIL(SB_ERR_ARG, "sb_conv_heads: %d channels in rows of %d", channels, ld);
+  HeadsArgs a;
+  a.proj = proj; a.n_rows = n_rows; a.ld = ld; a.hq = n_q_heads; a.hkv = n_kv_heads; a.dim = dim; a.vdim = vdim; a.hd = hd;
+  a.w = w; a.row_seq = row_seq; a.row_pos = row_pos; a.seq_pos0 = seq_pos0; a.seq_slot = seq_slot; a.page_off = page_off;
+  a.page_ids = page_ids; a.page_size = page_size; a.state = taps > 1 ? state : nullptr; a.cache = cache; a.q_out = q_out;
+  const bool own = n_rows == n_seqs;
+  const bool vec = dim % 4 == 0 && vdim % 4 == 0 && hd % 4 == 0 && ld % 4 == 0 &&
+                   (((uintptr_t)proj | (uintptr_t)state | (uintptr_t)cache | (uintptr_t)q_out) & 15) == 0;
+  SB_DISPATCH_DTYPE(w_dtype, TW, {
+    SB_DISPATCH_DTYPE(dtype, T, {
+      switch (taps) {
+        case 1: launch_conv_heads<1, TW, T>(a, own, vec, stream); break;
+        case 2: launch_conv_heads<2, TW, T>(a, own, vec, stream); break;
+        case 3: launch_conv_heads<3, TW, T>(a, own, vec, stream); break;
+        case 4: launch_conv_heads<4, TW, T>(a, own, vec, stream); break;
+        default: launch_conv_heads<5, TW, T>(a, own, vec, stream); break;
+      }
+    });
+  });
+  SB_CHECK_LAUNCH("sb_conv_heads");
+  if (!own && taps > 1) {
+    sb_launch<SB_K_ELEMENTWISE>(conv_state_kernel, dim3(n_seqs, (channels + 255) / 256), dim3(256), 0, stream, proj, ld, 0,
+                                channels, taps, seq_row0, seq_slot, state);
+    SB_CHECK_LAUNCH("sb_conv_heads (state)");
   }
   return SB_OK;
 }

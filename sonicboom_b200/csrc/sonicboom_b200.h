@@ -35,9 +35,15 @@ enum SbStatus { SB_OK = 0, SB_ERR_ARG = 1, SB_ERR_UNSUPPORTED = 2, SB_ERR_CUDA =
 /* What a product does with its finished rows.  SB_EPI_SWIGLU: the weight's rows alternate in
  * blocks of 8 (8 gate rows, the 8 up rows of the same outputs); out[m, o] = silu(gate) * up and
  * has N / 2 columns. */
-enum SbEpilogue { SB_EPI_NONE = 0, SB_EPI_BIAS = 1, SB_EPI_RESIDUAL = 2, SB_EPI_SWIGLU = 3 };
+enum SbEpilogue { SB_EPI_NONE = 0, SB_EPI_BIAS = 1, SB_EPI_RESIDUAL = 2, SB_EPI_SWIGLU = 3,
+                  SB_EPI_RELU2 = 4 /* the square of relu */ };
 /* The activation of a gated feed-forward: act(gate) * up. */
 enum SbGate { SB_GATE_SILU = 0, SB_GATE_CLAMPED = 1, SB_GATE_GELU_TANH = 2 };
+/* The activation of an expert: the clamped gated form of gate and up, or the square of relu of up alone. */
+enum SbExpert { SB_EXPERT_CLAMPED = 0, SB_EXPERT_RELU2 = 1 };
+/* What a row kernel writes along with a finished row: nothing, the row's RMS norm, the row itself, its
+ * layer norm. */
+enum SbNext { SB_NEXT_NONE = 0, SB_NEXT_RMS = 1, SB_NEXT_COPY = 2, SB_NEXT_LAYER = 3 };
 /* Kernel classes: bits of the mask that says which kernels are launched with programmatic
  * dependent launch (sb_set_pdl). */
 enum SbKernelClass {
@@ -177,6 +183,18 @@ int sb_glu_clamped(const float* gu, int n_rows, int ff, float limit, float alpha
 int sb_gated_act(const float* gu, int n_rows, int ff, int kind, float limit, float alpha, int interleaved,
                  void* out, int out_dtype, sb_stream_t stream);
 int sb_scale(float* x, size_t n, float c, sb_stream_t stream);          /* x *= c */
+/* out[r] = x[r] + w * y[r], or with norm_y x[r] + w * y[r] / sqrt(mean(y[r]^2) + eps) (w has `width`
+ * values; out may be x).  next (SbNext): next_out receives the finished row's RMS norm (next_w, next_eps),
+ * the row itself, or its layer norm (next_w, optionally next_b, next_eps), in next_out_dtype. */
+int sb_stream_join(const float* y, const float* x, int n_rows, int width, const void* w, int w_dtype,
+                   int norm_y, float eps, float* out, int next, const void* next_w,
+                   const void* next_b, int next_w_dtype, float next_eps, void* next_out,
+                   int next_out_dtype, sb_stream_t stream);
+/* out[r, c] = gelu(z[r * z_ld + c]) * table[tokens[r] * ld + at + c], c < dim, gelu in its tanh form; an id
+ * outside the table gives NaN. */
+int sb_side_gate(const float* z, int z_ld, int n_rows, int dim, const int32_t* tokens, const void* table,
+                 int table_dtype, int vocab, int ld, int at, void* out, int out_dtype,
+                 sb_stream_t stream);
 
 /* ---- attention over a cached latent ----
  * proj[r] = [n_heads x (dim | rd) | rank | rd] (the last two only with has_kv).  Rotates the first
@@ -214,12 +232,15 @@ int sb_mlstm_out(const float* num, const float* m_row, const float* proj, int n_
                  int out_dtype, sb_stream_t stream);
 
 /* Plain attention over the paged cache (float32 arithmetic, any head size up to 1024).  sink: null,
- * or one float32 per query head whose exponential joins that head's softmax denominator. */
+ * or one float32 per query head whose exponential joins that head's softmax denominator.  chunk > 0: key
+ * j is visible at position i only when j / chunk = i / chunk (whole parts).  bias: null, or float32
+ * [n_q_heads][bias_len] added to the capped score by distance, the last entry for all larger ones. */
 int sb_attention_plain(const void* q, void* out, int act_dtype, int n_rows, const int32_t* row_seq,
                        const int32_t* row_pos, const int32_t* page_off, const int32_t* page_ids,
                        int page_size, const void* cache, int cache_dtype, int n_q_heads,
                        int n_kv_heads, int hd, int window, float scale, const float* sink,
-                       float softcap, sb_stream_t stream);
+                       float softcap, int chunk, const float* bias, int bias_len,
+                       sb_stream_t stream);
 
 /* ---- the stream, the feed-forward and mixers with projections of their own kind ----
  * out[r] = x[r] + add[r] + vec (add [rows, width] float32 and vec [width] are optional; out may be
@@ -291,9 +312,10 @@ int sb_embed_pair(const int32_t* tokens, int n_rows, const int32_t* row_seq, con
                   int mul_prev, int mul_cur, int width, float scale, float* out, sb_stream_t stream);
 int sb_keep_last_token(const int32_t* tokens, const int32_t* seq_row0, const int32_t* seq_slot,
                        int n_seqs, int32_t* prev_token, sb_stream_t stream);
-/* out[r] = (x - mean) / sqrt(var + eps) * weight over the row x[rows ? rows[r] : r] */
+/* out[r] = (x - mean) / sqrt(var + eps) * weight [+ bias] over the row x[rows ? rows[r] : r]; the
+ * optional bias has the weight's dtype. */
 int sb_layernorm(const float* x, const int32_t* rows, int n_rows, int width, const void* weight,
-                 int weight_dtype, float eps, void* out, int out_dtype, sb_stream_t stream);
+                 const void* bias, int weight_dtype, float eps, void* out, int out_dtype, sb_stream_t stream);
 /* out[r, out_off + c] = act([x_t +] [bias +] sum_j w[c, j] x_(t - taps + 1 + j)) over the `channels`
  * columns of x at x_off; taps before a step's first row of a sequence come from state [slot,
  * taps - 1, channels] (float32), which then receives the step's last taps - 1 inputs; act 1: silu. */
@@ -302,6 +324,18 @@ int sb_causal_conv(const float* x, int n_rows, int ld, int x_off, int channels, 
                    const int32_t* row_seq, const int32_t* row_pos, const int32_t* seq_row0,
                    const int32_t* seq_pos0, const int32_t* seq_slot, float* state, void* out,
                    int out_dtype, int ld_out, int out_off, sb_stream_t stream);
+
+/* The convolution of sb_causal_conv (no bias, no activation) over the fused projection rows [q: n_q_heads
+ * x dim | k: n_kv_heads x dim | v: n_kv_heads x vdim], w [channels, taps] in that order, with the results
+ * written to q_out [rows, n_q_heads, hd] and to the pages of each row's position, padded with zeros to
+ * hd; both in `dtype`.  state [slot, taps - 1, channels]; at most sb_conv_heads_max_taps() taps. */
+int sb_conv_heads(const float* proj, int n_rows, int ld, int n_q_heads, int n_kv_heads, int dim, int vdim,
+                  int hd, int taps, const void* w, int w_dtype, int n_seqs, const int32_t* row_seq,
+                  const int32_t* row_pos, const int32_t* seq_row0, const int32_t* seq_pos0,
+                  const int32_t* seq_slot, const int32_t* page_off, const int32_t* page_ids,
+                  int page_size, float* state, void* cache, void* q_out, int dtype,
+                  sb_stream_t stream);
+int sb_conv_heads_max_taps(void);
 
 /* ---- the generalized delta rule ----
  * aux [rows, 3, n_heads * dim] = decays exp(-decay_scale * sigmoid(w2 . tanh(proj[z_off : z_off + rank])
@@ -345,23 +379,34 @@ int sb_moe_route(const float* logits, int n_rows, int n_experts, int top, int32_
  * lie in n_groups equal groups of neighbours, a group's score is the sum of its group_top largest
  * choice scores, and only experts of the keep_groups best groups can be chosen; the `top` largest
  * choice scores win (the lower index on a tie); weights s * scale, over the chosen ones' sum of s
- * first when `renormalize`. */
-int sb_moe_route_scored(const float* logits, const float* correction, int n_rows, int n_experts, int top,
-                        int n_groups, int keep_groups, int group_top, float scale, int renormalize,
+ * (+ 1e-20) first when `renormalize`.  With `softmax` s is the softmax of the row's logits.  Rows of
+ * logits lie ld values apart. */
+int sb_moe_route_scored(const float* logits, int ld, const float* correction, int n_rows, int n_experts,
+                        int softmax, int top, int n_groups, int keep_groups, int group_top, float scale, int renormalize,
                         int32_t* ids, float* weights, sb_stream_t stream);
 /* Pairs of a tile of one expert (32, 64 or 128) that group, up and down of one step share. */
 int sb_moe_tile_rows(int dtype, int n_pairs, int n_experts, int ff, int width);
 int sb_moe_max_tiles(int n_pairs, int n_experts, int tile_rows);
+/* Ids from n_experts on belong to no expert and are left out of the grouping. */
 int sb_moe_group(const int32_t* ids, int n_pairs, int n_experts, int tile_rows, int32_t* order, int32_t* meta,
                  sb_stream_t stream);
+/* kind (SbExpert): the clamped gated form, or the square of relu (w then [experts, ff, width]). */
 int sb_moe_up(const void* a, int a_dtype, const void* w, int w_dtype, const int32_t* order,
               const int32_t* meta, int n_pairs, int n_experts, int tile_rows, int top, int ff, int width,
-              float limit, float slope, void* act, sb_stream_t stream);
+              int kind, float limit, float slope, void* act, sb_stream_t stream);
 int sb_moe_down(const void* act, int a_dtype, const void* w, int w_dtype, const int32_t* order,
                 const int32_t* meta, int n_pairs, int n_experts, int tile_rows, int top, int width, int ff,
                 float* pair_out, sb_stream_t stream);
 int sb_moe_combine(float* x, const float* pair_out, const float* weights, int n_rows, int top, int width,
                    sb_stream_t stream);
+
+/* x[r] += scale * (sum over the row's choices of weight * (the pair's row, or h[r] where the id is
+ * n_experts or more) + sigmoid(gate[r * gate_ld]) * shared[r]); scale [width], shared, gate (without it
+ * the shared row counts once) and copy (x[r] in copy_dtype) are optional. */
+int sb_moe_join(float* x, const float* pair_out, const int32_t* ids, const float* weights, int n_experts,
+                const void* h, int h_dtype, const float* shared, const float* gate, int gate_ld,
+                const void* scale, int scale_dtype, int n_rows, int top, int width, void* copy,
+                int copy_dtype, sb_stream_t stream);
 
 int sb_sample_params_size(void);
 int sb_sample(float* logits, int n_rows, int vocab, const void* params, const int32_t* history,
@@ -381,14 +426,14 @@ int sb_attention_last_launches(void);     /* kernels the last sb_attention call 
 size_t sb_attention_scratch_bytes(int n_rows, int n_q_heads, int n_kv_heads, int max_new,
                                   int max_len);
 /* Causal grouped-query attention of a step's rows over one cache entry's pages (bfloat16).
- * sink: as in sb_attention_plain. */
+ * sink, chunk, bias: as in sb_attention_plain. */
 int sb_attention(const void* q, void* out, int n_rows, int n_seqs, int max_new,
                  const int32_t* seq_row0, const int32_t* seq_pos0, const int32_t* page_off,
                  const int32_t* page_ids, int page_size, const void* cache, int n_q_heads,
                  int n_kv_heads, int hd, int window, float scale, void* scratch,
                  size_t scratch_bytes, int* counters, int n_counters, int max_len, int n_pages,
                  int n_sms, const void* warm, size_t warm_bytes, const float* sink, float softcap,
-                 sb_stream_t stream);
+                 int chunk, const float* bias, int bias_len, sb_stream_t stream);
 
 #ifdef __cplusplus
 }

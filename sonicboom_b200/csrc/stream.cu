@@ -4,6 +4,9 @@
 //   sb_norm_add:   out[r] = x[r] + y[r] / sqrt(mean(y[r]^2) + eps) * w
 //   sb_gated_act:  out = act(gate) * up over [gate | up] rows: silu, the clamped form, or the tanh form of gelu
 //   sb_scale:      x *= c
+//   sb_stream_join: out[r] = x[r] + w * (y[r], or y[r] / sqrt(mean(y[r]^2) + eps)), then optionally the RMS norm
+//                  or the layer norm of the finished row, or the row itself in another dtype
+//   sb_side_gate:  out[r] = gelu(z[r]) * the part [at, at + dim) of the row's token in a second table
 //   sb_depth_mix:  out[r] = sum_j c[j] * planes[j][r]           (j ascending, float32)
 //
 // Both can also deliver the RMS norm of the row they have just finished (the first norm of
@@ -196,6 +199,146 @@ __global__ void gated_act_kernel(const float* gu, size_t n, int ff, int kind, fl
   }
 }
 
+// A sublayer's result joins the stream times a weight per channel, normed first or not, and what reads the
+// finished row next is written along (`next`: SbNext).  With ITEMS > 0 a thread keeps its part of the row in
+// registers (rows of at most NT * ITEMS * 4 values, 16-byte accesses): y and x are read once and the layer
+// norm's two passes touch no memory.  ITEMS = 0 walks the row in memory, any width.
+template <int NT, int ITEMS, typename TW, typename TN, typename TO>
+__global__ void __launch_bounds__(NT)
+stream_join_kernel(const float* y, const float* x, int width, const TW* __restrict__ w, int norm_y, float eps, float* out,
+                   int next, const TN* __restrict__ next_w, const TN* __restrict__ next_b, float next_eps, TO* next_out) {
+  __shared__ float red[NT / 32 + 1];
+  sb_pdl_launch();
+  const size_t r = blockIdx.x;
+  const float* yr = y + r * width;
+  const float* xr = x + r * width;
+  float* o = out + r * width;
+  TO* no = next_out + (next == SB_NEXT_NONE ? 0 : r * width);
+  const float n = (float)width;
+  if constexpr (ITEMS > 0) {
+    Vec<4> v[ITEMS];
+    float wv[ITEMS][4];
+#pragma unroll
+    for (int i = 0; i < ITEMS; ++i) {              // the weights wait for nobody
+      const int e = (threadIdx.x + i * NT) * 4;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) wv[i][j] = e < width ? sb_to_f32<TW>(w[e + j]) : 0.0f;
+    }
+    sb_pdl_wait();
+    float s = 0.0f;
+#pragma unroll
+    for (int i = 0; i < ITEMS; ++i) {
+      const int e = (threadIdx.x + i * NT) * 4;
+      if (e < width) {
+        v[i] = ld<4>(yr + e);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) s = fmaf(v[i].v[j], v[i].v[j], s);
+      }
+    }
+    const float inv = norm_y ? 1.0f / sqrtf(block_sum<NT>(s, red) / n + eps) : 1.0f;
+    float sum = 0.0f, sq = 0.0f;
+#pragma unroll
+    for (int i = 0; i < ITEMS; ++i) {
+      const int e = (threadIdx.x + i * NT) * 4;
+      if (e < width) {
+        const Vec<4> b = ld<4>(xr + e);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          v[i].v[j] = b.v[j] + (v[i].v[j] * inv) * wv[i][j];
+          sum += v[i].v[j];
+          sq = fmaf(v[i].v[j], v[i].v[j], sq);
+        }
+        st<4>(o + e, v[i]);
+      }
+    }
+    if (next == SB_NEXT_NONE) return;
+    float mean = 0.0f, nv = 1.0f;
+    if (next == SB_NEXT_LAYER) {
+      mean = block_sum<NT>(sum, red) / n;
+      sq = 0.0f;
+#pragma unroll
+      for (int i = 0; i < ITEMS; ++i) {
+        if ((threadIdx.x + i * NT) * 4 < width) {
+#pragma unroll
+          for (int j = 0; j < 4; ++j) {
+            const float d = v[i].v[j] - mean;
+            sq = fmaf(d, d, sq);
+          }
+        }
+      }
+    }
+    if (next != SB_NEXT_COPY) nv = 1.0f / sqrtf(block_sum<NT>(sq, red) / n + next_eps);
+#pragma unroll
+    for (int i = 0; i < ITEMS; ++i) {
+      const int e = (threadIdx.x + i * NT) * 4;
+      if (e < width) {
+        float t[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          t[j] = v[i].v[j];
+          if (next != SB_NEXT_COPY) t[j] = ((t[j] - mean) * nv) * sb_to_f32<TN>(next_w[e + j]);
+          if (next_b) t[j] += sb_to_f32<TN>(next_b[e + j]);
+        }
+        if constexpr (sizeof(TO) == 2) {
+          __nv_bfloat162 a = __floats2bfloat162_rn(t[0], t[1]), b = __floats2bfloat162_rn(t[2], t[3]);
+          uint2 u;
+          u.x = *reinterpret_cast<uint32_t*>(&a);
+          u.y = *reinterpret_cast<uint32_t*>(&b);
+          *reinterpret_cast<uint2*>(no + e) = u;
+        } else {
+#pragma unroll
+          for (int j = 0; j < 4; ++j) no[e + j] = sb_from_f32<TO>(t[j]);
+        }
+      }
+    }
+  } else {
+    sb_pdl_wait();
+    float s = 0.0f;
+    if (norm_y)
+      for (int i = threadIdx.x; i < width; i += NT) s = fmaf(yr[i], yr[i], s);
+    const float inv = norm_y ? 1.0f / sqrtf(block_sum<NT>(s, red) / n + eps) : 1.0f;
+    float sum = 0.0f, sq = 0.0f;
+    for (int i = threadIdx.x; i < width; i += NT) {
+      const float v = xr[i] + (yr[i] * inv) * sb_to_f32<TW>(w[i]);
+      o[i] = v;
+      sum += v;
+      sq = fmaf(v, v, sq);
+    }
+    if (next == SB_NEXT_NONE) return;
+    float mean = 0.0f, nv = 1.0f;
+    if (next == SB_NEXT_LAYER) {
+      mean = block_sum<NT>(sum, red) / n;
+      sq = 0.0f;
+      for (int i = threadIdx.x; i < width; i += NT) {        // a thread reads back what it wrote itself
+        const float d = o[i] - mean;
+        sq = fmaf(d, d, sq);
+      }
+    }
+    if (next != SB_NEXT_COPY) nv = 1.0f / sqrtf(block_sum<NT>(sq, red) / n + next_eps);
+    for (int i = threadIdx.x; i < width; i += NT) {
+      float t = o[i];
+      if (next != SB_NEXT_COPY) t = ((t - mean) * nv) * sb_to_f32<TN>(next_w[i]);
+      if (next_b) t += sb_to_f32<TN>(next_b[i]);
+      no[i] = sb_from_f32<TO>(t);
+    }
+  }
+}
+
+// One thread per value: gelu(z) in its tanh form times the token's entry in the table (a row of `ld` values;
+// this layer's part starts at `at`).  An id outside the table gives NaN.
+template <typename TT, typename TO>
+__global__ void side_gate_kernel(const float* z, int z_ld, const int32_t* tokens, const TT* __restrict__ table, int vocab, int ld,
+                                 int at, size_t n, int dim, TO* out) {
+  sb_pdl_launch();
+  sb_pdl_wait();
+  for (size_t e = (size_t)blockIdx.x * blockDim.x + threadIdx.x; e < n; e += (size_t)gridDim.x * blockDim.x) {
+    const size_t r = e / dim, c = e % dim;
+    const int tok = tokens[r];
+    const float t = (unsigned)tok < (unsigned)vocab ? sb_to_f32<TT>(table[(size_t)tok * ld + at + c]) : __int_as_float(0x7fc00000);
+    out[e] = sb_from_f32<TO>(sb_gelu_tanh(z[r * z_ld + c]) * t);
+  }
+}
+
 __global__ void scale_kernel(float* x, size_t n, float c) {
   sb_pdl_launch();
   sb_pdl_wait();
@@ -317,5 +460,56 @@ extern "C" int sb_scale(float* x, size_t n, float c, cudaStream_t stream) {
   const int blocks = (int)((n + 255) / 256 < 8192 ? (n + 255) / 256 : 8192);
   sb_launch<SB_K_ELEMENTWISE>(scale_kernel, dim3(blocks), dim3(256), 0, stream, x, n, c);
   SB_CHECK_LAUNCH("sb_scale");
+  return SB_OK;
+}
+
+extern "C" int sb_stream_join(const float* y, const float* x, int n_rows, int width, const void* w, int w_dtype, int norm_y,
+                              float eps, float* out, int next, const void* next_w, const void* next_b, int next_w_dtype,
+                              float next_eps, void* next_out, int next_out_dtype, cudaStream_t stream) {
+  if (n_rows <= 0 || width <= 0 || !y || !x || !w || !out) SB_FAIL(SB_ERR_ARG, "sb_stream_join: rows=%d width=%d", n_rows, width);
+  const bool has_next = next != SB_NEXT_NONE, normed = next == SB_NEXT_RMS || next == SB_NEXT_LAYER;
+  if (next < SB_NEXT_NONE || next > SB_NEXT_LAYER || (has_next && !next_out) || (normed && !next_w) || (!normed && next_b))
+    SB_FAIL(SB_ERR_ARG, "sb_stream_join: what comes next (%d) does not fit its arguments", next);
+  if (!sb_valid_dtype(w_dtype) || (has_next && !sb_valid_dtype(next_out_dtype)) || (normed && !sb_valid_dtype(next_w_dtype)))
+    SB_FAIL(SB_ERR_ARG, "sb_stream_join: dtype codes %d %d %d", w_dtype, next_w_dtype, next_out_dtype);
+  if (!(eps >= 0.0f) || !(next_eps >= 0.0f)) SB_FAIL(SB_ERR_ARG, "sb_stream_join: eps %g %g", eps, next_eps);
+  const bool vec = width % 4 == 0 && (((uintptr_t)y | (uintptr_t)x | (uintptr_t)out | (uintptr_t)next_out) & 15) == 0;
+#define SB_JOIN(NT, ITEMS)                                                                                               \
+  sb_launch<SB_K_ELEMENTWISE>(stream_join_kernel<NT, ITEMS, TW, TN, TO>, dim3(n_rows), dim3(NT), 0, stream, y, x, width,  \
+                              (const TW*)w, norm_y, eps, out, next, (const TN*)next_w, (const TN*)next_b, next_eps,       \
+                              (TO*)next_out)
+  SB_DISPATCH_DTYPE(w_dtype, TW, {
+    SB_DISPATCH_NEXT(normed, next_w_dtype, TN, {
+      SB_DISPATCH_NEXT(has_next, next_out_dtype, TO, {
+        if (!vec || width > 16384) SB_JOIN(256, 0);
+        else if (width <= 1024) SB_JOIN(256, 1);
+        else if (n_rows <= 256 && width <= 4096) SB_JOIN(1024, 1);      // few rows: a row's loads in flight together
+        else if (width <= 2048) SB_JOIN(256, 2);
+        else if (width <= 4096) SB_JOIN(256, 4);
+        else if (width <= 8192) SB_JOIN(512, 4);
+        else SB_JOIN(1024, 4);
+      });
+    });
+  });
+#undef SB_JOIN
+  SB_CHECK_LAUNCH("sb_stream_join");
+  return SB_OK;
+}
+
+extern "C" int sb_side_gate(const float* z, int z_ld, int n_rows, int dim, const int32_t* tokens, const void* table, int table_dtype,
+                            int vocab, int ld, int at, void* out, int out_dtype, cudaStream_t stream) {
+  if (n_rows <= 0 || dim <= 0 || vocab <= 0 || !z || !tokens || !table || !out || at < 0 || at + dim > ld || z_ld < dim)
+    SB_FAIL(SB_ERR_ARG, "sb_side_gate: rows=%d dim=%d at %d of %d", n_rows, dim, at, ld);
+  if (!sb_valid_dtype(table_dtype) || !sb_valid_dtype(out_dtype))
+    SB_FAIL(SB_ERR_ARG, "sb_side_gate: dtype codes %d %d", table_dtype, out_dtype);
+  const size_t n = (size_t)n_rows * dim;
+  const int blocks = (int)((n + 255) / 256 < 8192 ? (n + 255) / 256 : 8192);
+  SB_DISPATCH_DTYPE(table_dtype, TT, {
+    SB_DISPATCH_DTYPE(out_dtype, TO, {
+      sb_launch<SB_K_ELEMENTWISE>(side_gate_kernel<TT, TO>, dim3(blocks), dim3(256), 0, stream, z, z_ld, tokens,
+                                  (const TT*)table, vocab, ld, at, n, dim, (TO*)out);
+    });
+  });
+  SB_CHECK_LAUNCH("sb_side_gate");
   return SB_OK;
 }

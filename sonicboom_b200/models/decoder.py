@@ -44,7 +44,7 @@ class DecoderModel:
         # what joins the stream right before a schedule entry: {entry: StreamInjection}
         self.injections = {inj.before_entry: inj for inj in spec.injections}
         self.injection_vectors = {}
-        self.embedding = self.head = self.pair_table = None
+        self.embedding = self.head = self.pair_table = self.side_table = None
 
     # ------------------------------------------------------------------ weights
     def tensor_requests(self) -> list[TensorRequest]:
@@ -57,6 +57,8 @@ class DecoderModel:
         req += self.final_norm.tensor_requests()
         if s.pair_embedding is not None:
             req.append(TensorRequest(s.pair_embedding.tensor, (s.pair_embedding.buckets + 1, s.width), "embedding"))
+        if s.side_table is not None:
+            req.append(TensorRequest(s.side_table.tensor, (s.vocab, s.side_table.parts * s.side_table.dim), "embedding"))
         req += [TensorRequest(inj.tensor, (inj.rows, s.width), "bias") for inj in s.injections if inj.tensor]
         req += [TensorRequest(name, tuple(shape), optional=True) for name, shape in s.unused_tensors]
         if s.head_tensor is not None:
@@ -72,6 +74,8 @@ class DecoderModel:
             self.pair_table = get(self.spec.pair_embedding.tensor)
             if self.pair_table.dtype != self.embedding.dtype:
                 self.pair_table, self.embedding = self.pair_table.float(), self.embedding.float()
+        if self.spec.side_table is not None:
+            self.side_table = get(self.spec.side_table.tensor)
         for b, m in zip(self.blocks, self.depth_mixes):
             b.bind(get)
             if m is not None:
@@ -98,7 +102,8 @@ class DecoderModel:
             mine, own = self.blocks[e.layer].kv_need(), needs[e.cache_from]
             window = 0 if 0 in (mine.window, own.window) else max(mine.window, own.window)
             needs[e.cache_from] = KVNeed(own.n_kv_heads, own.head_dim, window,
-                                         max(mine.keep_first, own.keep_first) if window else 0)
+                                         max(mine.keep_first, own.keep_first) if window else 0,
+                                         own.chunk if mine.chunk == own.chunk else 0)
         return needs
 
     def state_needs(self) -> list:
@@ -123,7 +128,7 @@ class DecoderModel:
             if any(m is not None for m in mixes) else None
         x = streams[0] if streams is not None else \
             torch.empty((plan.n_rows, s.width), dtype=torch.float32, device=self.device)
-        ctx = StepContext(plan=plan, cache=cache)
+        ctx = StepContext(plan=plan, cache=cache, side_table=self.side_table)
         if s.pair_embedding is None:
             ops.embed(plan.tokens, self.embedding, x, s.embedding_scale)
         else:

@@ -15,7 +15,7 @@ from . import abi as _abi
 from .csrc import build as _build
 
 F32, BF16 = 0, 1
-EPI_NONE, EPI_BIAS, EPI_RESIDUAL, EPI_SWIGLU = 0, 1, 2, 3
+EPI_NONE, EPI_BIAS, EPI_RESIDUAL, EPI_SWIGLU, EPI_RELU2 = 0, 1, 2, 3, 4
 SWIGLU_BLOCK = 8                 # rows of gate and up alternate in blocks of this many
 SKINNY_MAX_ROWS = 64             # bfloat16 products of at most this many rows stream the weights
 DECODE_ATTENTION_ROWS = 16       # query rows (new tokens x heads) of one key/value head that the split decode attention takes
@@ -190,6 +190,8 @@ def linear(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int = 
     places (inside the tcgen05 and the weight-streaming kernels, else the plain product followed by
     `gated_act`).
 
+    EPI_RELU2 stores max(v, 0)^2, in every kernel.
+
     `norm` = (weight, eps, norm_out) also writes norm_out = rmsnorm(out, weight, eps) [M,N]
     (out must be float32): in the kernel that finishes the product where one does (the split-K
     decode form of the tcgen05 kernel), else with the norm kernel after it.
@@ -242,7 +244,7 @@ def linear(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int = 
     l = lib()
     if norm is not None:
         norm_w, norm_eps, norm_out = norm
-        assert out.dtype == torch.float32 and epilogue != EPI_SWIGLU
+        assert out.dtype == torch.float32 and epilogue not in (EPI_SWIGLU, EPI_RELU2)
         assert norm_w.numel() == N and tuple(norm_out.shape) == (M, N)
         fuses = fast and kernel in ("auto", "tc5") and bool(l.sb_gemm_tc5_fuses_norm(
             M, N, K, _sm_count(a.device), epilogue, _code(out.dtype), 0))
@@ -500,10 +502,14 @@ def attention_lib(head_dim: int):
 def attention(q: torch.Tensor, out: torch.Tensor, plan, group_index: int, cache: torch.Tensor,
               n_q_heads: int, n_kv_heads: int, head_dim: int, window: int, scale: float,
               kernel: str = "auto", warm: torch.Tensor | None = None,
-              sink: torch.Tensor | None = None, softcap: float = 0.0) -> torch.Tensor:
+              sink: torch.Tensor | None = None, softcap: float = 0.0, chunk: int = 0,
+              bias: torch.Tensor | None = None) -> torch.Tensor:
     """Causal grouped-query attention of the step's rows over one cache entry's pages.
     `sink` (float32, one per query head): exp(sink) joins that head's softmax denominator.
     `softcap` c > 0: a score s becomes c tanh(s / c) before the softmax.
+    `chunk` c > 0: only keys of the query's own stretch of c positions, counted from the sequence's
+    start, are visible.  `bias` (float32 [query heads, n]): the capped score of a key d positions back
+    gets bias[h, min(d, n - 1)] added.
 
     bfloat16 runs the tensor-core kernels (built for the head size at first use); float32, a
     head size those kernels do not take, or `kernel="plain"` run the plain kernel.  `"mma"` keeps
@@ -516,6 +522,9 @@ def attention(q: torch.Tensor, out: torch.Tensor, plan, group_index: int, cache:
     g = plan.groups[group_index]
     if sink is not None:
         assert sink.dtype == torch.float32 and sink.numel() == n_q_heads
+    if bias is not None:
+        assert bias.dtype == torch.float32 and bias.dim() == 2 and bias.shape[0] == n_q_heads
+    bias_len = bias.shape[1] if bias is not None else 0
     al = attention_lib(head_dim) if (q.dtype == torch.bfloat16 and cache.dtype == torch.bfloat16
                                      and kernel != "plain") else None
     if al is not None:
@@ -531,7 +540,7 @@ def attention(q: torch.Tensor, out: torch.Tensor, plan, group_index: int, cache:
             head_dim, window, ctypes.c_float(scale), _ptr(scratch),
             ctypes.c_size_t(scratch.numel() if scratch is not None else 0),
             _ptr(counters), counters.numel(), plan.max_len, cache.shape[0], _sm_count(q.device),
-            *_warm_args(warm), _ptr(sink), ctypes.c_float(softcap), _stream())
+            *_warm_args(warm), _ptr(sink), ctypes.c_float(softcap), int(chunk), _ptr(bias), bias_len, _stream())
         if kernel in ("mma", "tma"):
             al.sb_attention_force_mma({"mma": 1, "tma": 2}.get(_os.environ.get("SB_ATTN", ""), 0))
         if rc != 0:
@@ -544,7 +553,7 @@ def attention(q: torch.Tensor, out: torch.Tensor, plan, group_index: int, cache:
             _i32(plan.row_pos, "row_pos"), _i32(g.page_off, "page_off"),
             _i32(g.page_ids, "page_ids"), g.page_size, _ptr(cache), _code(cache.dtype),
             n_q_heads, n_kv_heads, head_dim, window, ctypes.c_float(scale), _ptr(sink),
-            ctypes.c_float(softcap), _stream()), "attention (plain kernel)")
+            ctypes.c_float(softcap), int(chunk), _ptr(bias), bias_len, _stream()), "attention (plain kernel)")
     return out
 
 
@@ -663,6 +672,38 @@ def norm_add(y: torch.Tensor, x: torch.Tensor, weight: torch.Tensor, eps: float,
     _check(lib().sb_norm_add(_ptr(y), _ptr(x), rows, width, _ptr(weight), _code(weight.dtype),
                              ctypes.c_float(eps), _ptr(out), *_next_norm_args(next_norm, width, rows),
                              _stream()), "norm_add")
+    return out
+
+
+NEXT_NONE, NEXT_RMS, NEXT_COPY, NEXT_LAYER = 0, 1, 2, 3
+
+
+def stream_join(y: torch.Tensor, x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor,
+                norm_eps: float | None = None, then: tuple | None = None) -> torch.Tensor:
+    """out = x + weight * y row by row in float32 (out may be x); with `norm_eps` y is divided by its
+    root mean square first, sqrt(mean(y^2) + norm_eps).  `then` also writes what reads the finished rows
+    next: (NEXT_RMS, weight, None, eps, out), (NEXT_LAYER, weight, bias or None, eps, out) or
+    (NEXT_COPY, None, None, 0.0, out), in that tensor's dtype."""
+    rows, width = y.shape
+    assert y.dtype == x.dtype == out.dtype == torch.float32 and x.shape == y.shape == out.shape
+    assert weight.numel() == width
+    kind, w, b, eps, nxt = then if then is not None else (NEXT_NONE, None, None, 0.0, None)
+    assert nxt is None or tuple(nxt.shape) == (rows, width)
+    assert w is None or (w.numel() == width and (b is None or (b.numel() == width and b.dtype == w.dtype)))
+    _check(lib().sb_stream_join(_ptr(y), _ptr(x), rows, width, _ptr(weight), _code(weight.dtype),
+                                0 if norm_eps is None else 1, ctypes.c_float(norm_eps or 0.0), _ptr(out), kind, _ptr(w),
+                                _ptr(b), _code(w.dtype) if w is not None else 0, ctypes.c_float(eps), _ptr(nxt),
+                                _code(nxt.dtype) if nxt is not None else 0, _stream()), "stream_join")
+    return out
+
+
+def side_gate(z: torch.Tensor, tokens: torch.Tensor, table: torch.Tensor, at: int, out: torch.Tensor) -> torch.Tensor:
+    """out[r] = gelu(z[r]) (tanh form) * table[tokens[r], at : at + dim], dim = out's width; z float32."""
+    rows, dim = out.shape
+    assert z.dtype == torch.float32 and z.shape[0] == rows == tokens.numel() and z.shape[1] >= dim
+    _check(lib().sb_side_gate(_ptr(z), z.shape[1], rows, dim, _i32(tokens, "tokens"), _ptr(table), _code(table.dtype),
+                              table.shape[0], table.shape[1], int(at), _ptr(out), _code(out.dtype), _stream()),
+           "side_gate")
     return out
 
 
@@ -974,13 +1015,14 @@ def keep_last_token(plan, prev_token: torch.Tensor) -> None:
 
 
 def layernorm(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor,
-              rows: torch.Tensor | None = None) -> torch.Tensor:
-    """out[r] = (x - mean) / sqrt(var + eps) * weight over the row x[rows[r]] or x[r] (no bias)."""
+              rows: torch.Tensor | None = None, bias: torch.Tensor | None = None) -> torch.Tensor:
+    """out[r] = (x - mean) / sqrt(var + eps) * weight [+ bias] over the row x[rows[r]] or x[r]."""
     assert x.dtype == torch.float32 and x.dim() == 2
     n, width = out.shape[0], x.shape[1]
     assert out.shape[1] == width and weight.numel() == width and (rows is not None or x.shape[0] == n)
+    assert bias is None or (bias.numel() == width and bias.dtype == weight.dtype)
     _check(lib().sb_layernorm(_ptr(x), _i32(rows, "rows") if rows is not None else _ptr(None), n, width,
-                              _ptr(weight), _code(weight.dtype), ctypes.c_float(eps), _ptr(out), _code(out.dtype),
+                              _ptr(weight), _ptr(bias), _code(weight.dtype), ctypes.c_float(eps), _ptr(out), _code(out.dtype),
                               _stream()), "layernorm")
     return out
 
@@ -1007,6 +1049,32 @@ def causal_conv(x: torch.Tensor, x_off: int, channels: int, w: torch.Tensor, bia
                                 out.shape[1], out_off, _stream()), "causal_conv",
            launches=1 if own or taps == 1 else 2)
     return out
+
+
+def conv_heads(proj: torch.Tensor, w: torch.Tensor, plan, page_off, page_ids, page_size: int, n_q_heads: int,
+               n_kv_heads: int, dim: int, vdim: int, state: torch.Tensor | None, cache: torch.Tensor,
+               q_out: torch.Tensor) -> torch.Tensor:
+    """`causal_conv` over the fused float32 projection rows [q | k | v] (w [channels, taps]) with its
+    results written as queries into q_out [rows, heads, head size] and as keys and values into the pages
+    of each row's position, heads padded with zeros.  At most `conv_heads_max_taps()` taps."""
+    n, ld = proj.shape
+    channels, taps = w.shape
+    assert proj.dtype == torch.float32 and channels == n_q_heads * dim + n_kv_heads * (dim + vdim) <= ld
+    assert q_out.dtype == cache.dtype and tuple(q_out.shape[:2]) == (n, n_q_heads)
+    if taps > 1:
+        assert state.dtype == torch.float32 and tuple(state.shape[1:]) == (taps - 1, channels)
+    own = plan.n_rows == plan.n_seqs
+    _check(lib().sb_conv_heads(_ptr(proj), n, ld, n_q_heads, n_kv_heads, dim, vdim, q_out.shape[2], taps, _ptr(w),
+                               _code(w.dtype), plan.n_seqs, _i32(plan.row_seq, "row_seq"), _i32(plan.row_pos, "row_pos"),
+                               _i32(plan.seq_row0, "seq_row0"), _i32(plan.seq_pos0, "seq_pos0"),
+                               _i32(plan.seq_slot, "seq_slot"), _i32(page_off, "page_off"), _i32(page_ids, "page_ids"),
+                               page_size, _ptr(state) if taps > 1 else None, _ptr(cache), _ptr(q_out), _code(q_out.dtype),
+                               _stream()), "conv_heads", launches=1 if own or taps == 1 else 2)
+    return q_out
+
+
+def conv_heads_max_taps() -> int:
+    return int(lib().sb_conv_heads_max_taps())
 
 
 # ---------------------------------------------------------------------- the generalized delta rule
@@ -1101,31 +1169,36 @@ def moe_route(logits: torch.Tensor, top: int, ids: torch.Tensor, weights: torch.
 
 def moe_route_scored(logits: torch.Tensor, correction: torch.Tensor | None, top: int, ids: torch.Tensor,
                      weights: torch.Tensor, groups: tuple = (1, 1), group_top: int = 2, scale: float = 1.0,
-                     renormalize: bool = False) -> None:
-    """Per row of float32 logits: scores s = sigmoid(logits); the `top` experts with the largest
+                     renormalize: bool = False, scores: str = "sigmoid") -> None:
+    """Per row of float32 logits: scores s = sigmoid(logits), or with `scores` "softmax" their softmax
+    (a row's first values only, when `correction` has fewer than the row); the `top` experts with the largest
     choice scores s + correction (float32 [experts] or None; the lower index wins a tie) into ids, their
     s * scale (over the chosen ones' sum of s first when `renormalize`) into weights.  `groups` =
     (count, keep): the experts lie in `count` equal groups of neighbours, a group's score is the sum of
     its `group_top` largest choice scores, and only experts of the `keep` best groups can be chosen."""
-    n, e = logits.shape
-    assert logits.dtype == weights.dtype == torch.float32 and ids.dtype == torch.int32
-    assert tuple(ids.shape) == tuple(weights.shape) == (n, top)
-    assert correction is None or (correction.dtype == torch.float32 and correction.numel() == e)
-    _check(lib().sb_moe_route_scored(_ptr(logits), _ptr(correction), n, e, top, int(groups[0]), int(groups[1]),
+    n, ld = logits.shape
+    e = ld if correction is None else correction.numel()
+    assert logits.dtype == weights.dtype == torch.float32 and ids.dtype == torch.int32 and e <= ld
+    assert tuple(ids.shape) == tuple(weights.shape) == (n, top) and scores in ("sigmoid", "softmax")
+    assert correction is None or correction.dtype == torch.float32
+    _check(lib().sb_moe_route_scored(_ptr(logits), ld, _ptr(correction), n, e, 1 if scores == "softmax" else 0, top, int(groups[0]), int(groups[1]),
                                      int(group_top), ctypes.c_float(scale), 1 if renormalize else 0, _ptr(ids),
                                      _ptr(weights), _stream()), "moe_route_scored")
 
 
-def moe_experts(h: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_up: torch.Tensor,
-                w_down: torch.Tensor, limit: float, slope: float, x: torch.Tensor) -> torch.Tensor:
-    """x[r] += sum over the row's choices k of weights[r, k] * expert ids[r, k] applied to h[r]; an
-    expert is down (g * sigmoid(slope g) * (u + 1)), g = min(gate h, limit), u = clamp(up h, +-limit).
-    w_up [experts, 2 (gate, up), ff, width], w_down [experts, width, ff], both in h's dtype."""
+EXPERT_CLAMPED, EXPERT_RELU2 = 0, 1
+
+
+def _moe_pairs(h, ids, w_up, w_down, kind, limit, slope):
+    """The chosen experts applied to their rows: float32 [rows * top, width], one row per (row, choice) pair
+    (left as it is where the id names no expert).  w_up is [experts, 2 (gate, up), ff, width] for
+    EXPERT_CLAMPED and [experts, ff, width] for EXPERT_RELU2."""
     n, width = h.shape
     top = ids.shape[1]
-    n_experts, _, ff, _ = w_up.shape
-    assert tuple(w_up.shape) == (n_experts, 2, ff, width) and tuple(w_down.shape) == (n_experts, width, ff)
-    assert h.dtype == w_up.dtype == w_down.dtype and x.dtype == torch.float32 and tuple(x.shape) == (n, width)
+    n_experts, ff = w_up.shape[0], w_up.shape[-2]
+    want = (n_experts, 2, ff, width) if kind == EXPERT_CLAMPED else (n_experts, ff, width)
+    assert tuple(w_up.shape) == want and tuple(w_down.shape) == (n_experts, width, ff)
+    assert h.dtype == w_up.dtype == w_down.dtype
     pairs = n * top
     l = lib()
     order = torch.empty(pairs, dtype=torch.int32, device=h.device)
@@ -1135,9 +1208,46 @@ def moe_experts(h: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_up:
     pair_out = torch.empty((pairs, width), dtype=torch.float32, device=h.device)
     _check(l.sb_moe_group(_ptr(ids), pairs, n_experts, tile, _ptr(order), _ptr(meta), _stream()), "moe_group")
     _check(l.sb_moe_up(_ptr(h), _code(h.dtype), _ptr(w_up), _code(w_up.dtype), _ptr(order), _ptr(meta), pairs,
-                       n_experts, tile, top, ff, width, ctypes.c_float(limit), ctypes.c_float(slope), _ptr(act),
+                       n_experts, tile, top, ff, width, kind, ctypes.c_float(limit), ctypes.c_float(slope), _ptr(act),
                        _stream()), "moe_up")
     _check(l.sb_moe_down(_ptr(act), _code(act.dtype), _ptr(w_down), _code(w_down.dtype), _ptr(order), _ptr(meta),
                          pairs, n_experts, tile, top, width, ff, _ptr(pair_out), _stream()), "moe_down")
-    _check(l.sb_moe_combine(_ptr(x), _ptr(pair_out), _ptr(weights), n, top, width, _stream()), "moe_combine")
+    return pair_out
+
+
+def moe_experts(h: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_up: torch.Tensor,
+                w_down: torch.Tensor, limit: float, slope: float, x: torch.Tensor) -> torch.Tensor:
+    """x[r] += sum over the row's choices k of weights[r, k] * expert ids[r, k] applied to h[r]; an
+    expert is down (g * sigmoid(slope g) * (u + 1)), g = min(gate h, limit), u = clamp(up h, +-limit).
+    w_up [experts, 2 (gate, up), ff, width], w_down [experts, width, ff], both in h's dtype."""
+    n, width = h.shape
+    assert x.dtype == torch.float32 and tuple(x.shape) == (n, width)
+    pair_out = _moe_pairs(h, ids, w_up, w_down, EXPERT_CLAMPED, limit, slope)
+    _check(lib().sb_moe_combine(_ptr(x), _ptr(pair_out), _ptr(weights), n, ids.shape[1], width, _stream()), "moe_combine")
+    return x
+
+
+def moe_relu2_join(h: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor,
+                   x: torch.Tensor, shared: torch.Tensor | None = None, gate: tuple | None = None,
+                   scale: torch.Tensor | None = None, copy: torch.Tensor | None = None) -> torch.Tensor:
+    """x[r] += scale * (sum over the row's choices k of weights[r, k] * y_k + sigmoid(g_r) * shared[r]), y_k
+    being expert ids[r, k] applied to h[r], down (relu(up h)^2), or h[r] itself for an id from the number
+    of experts on.  w_up [experts, ff, width], w_down [experts, width, ff] in h's dtype.  Optional: `shared`
+    float32 rows, `gate` = (float32 rows, column) with the shared rows' g, `scale` [width], `copy`, which
+    receives the finished rows of x in its own dtype."""
+    n, width = h.shape
+    assert x.dtype == torch.float32 and tuple(x.shape) == (n, width)
+    assert shared is None or (shared.dtype == torch.float32 and tuple(shared.shape) == (n, width))
+    g_ptr, g_ld = None, 0
+    if gate is not None:
+        g, col = gate
+        assert g.dtype == torch.float32 and g.is_contiguous() and g.shape[0] == n and 0 <= col < g.shape[1]
+        g_ptr, g_ld = g.data_ptr() + 4 * col, g.shape[1]
+    assert scale is None or scale.numel() == width
+    assert copy is None or tuple(copy.shape) == (n, width)
+    pair_out = _moe_pairs(h, ids, w_up, w_down, EXPERT_RELU2, 0.0, 0.0)
+    _check(lib().sb_moe_join(_ptr(x), _ptr(pair_out), _ptr(ids), _ptr(weights), w_up.shape[0], _ptr(h), _code(h.dtype),
+                             _ptr(shared), g_ptr, g_ld, _ptr(scale), _code(scale.dtype) if scale is not None else 0, n,
+                             ids.shape[1], width, _ptr(copy), _code(copy.dtype) if copy is not None else 0, _stream()),
+           "moe_join")
     return x

@@ -53,6 +53,7 @@ class StepContext:
     block_out: Optional[torch.Tensor] = None            # where the caller wants the running block's result (a block may ignore it)
     block_mix: Optional[tuple] = None                   # (depth mix, streams, next norm) the caller runs on that result; a block may run it with its last add
     mixed_out: Optional[torch.Tensor] = None            # what that depth mix handed on, when the block ran it
+    side_table: Optional[torch.Tensor] = None           # the model's second embedding table for layers with a token input
 
     def linear(self, a, w, out, epilogue, residual=None, bias=None, act_dtype=None):
         """ops.linear into float32 `out`; when `next_norm` is an RMS norm with a plain weight,
@@ -114,6 +115,11 @@ class Norm(Part):
     def as_rms(self) -> Optional[tuple]:
         """(weight, eps) when the norm is y = x / sqrt(mean(x^2) + eps) * weight, else None:
         what a product kernel needs to apply it to its own result."""
+        return None
+
+    def as_layer(self) -> Optional[tuple]:
+        """(weight, bias or None, eps) when the norm is a layer norm, y = (x - mean) / sqrt(var + eps) *
+        weight + bias, else None: what `ops.stream_join` needs to apply it to the rows it finishes."""
         return None
 
 

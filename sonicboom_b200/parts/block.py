@@ -337,3 +337,137 @@ class OutputNormBlock(Block):
         ctx.next_norm = ctx.next_weights = None
         y = self.feed_forward.forward(f, ctx)
         return self._join(y, x, self.w2, self.feed_forward_post_norm.as_rms()[1], ctx, after)
+
+
+class SideInput(Part):
+    """A layer's token input: g = gelu(gate x) * e with e the layer's part of the token's row in the model's
+    side table, y = proj g.  `forward` returns y; the block adds y / sqrt(mean(y^2) + eps) * norm to the
+    stream (`weight`, `eps`).  It reads the stream itself, in the activation dtype (`reads`)."""
+
+    def __init__(self, spec, dtype):
+        from .norm import StreamCast
+        self.spec, self.dtype, self.eps = spec, dtype, float(spec.eps)
+        self.reads = StreamCast()
+        self.w_gate = self.w_proj = self.weight = None
+
+    def tensor_requests(self):
+        s = self.spec
+        return [TensorRequest(s.prefix + "gate", (s.dim, s.width)), TensorRequest(s.prefix + "proj", (s.width, s.dim)),
+                TensorRequest(s.prefix + "norm", (s.width,), "norm")]
+
+    def bind(self, get):
+        p = self.spec.prefix
+        self.w_gate, self.w_proj, self.weight = get(p + "gate"), get(p + "proj"), get(p + "norm")
+
+    def forward(self, xc, ctx):
+        rows, s = xc.shape[0], self.spec
+        z = torch.empty((rows, s.dim), dtype=torch.float32, device=xc.device)
+        ops.linear(xc, self.w_gate, z)
+        g = torch.empty((rows, s.dim), dtype=self.dtype, device=xc.device)
+        ops.side_gate(z, ctx.plan.tokens, ctx.side_table, s.part * s.dim, g)
+        y = torch.empty((rows, s.width), dtype=torch.float32, device=xc.device)
+        return ops.linear(g, self.w_proj, y)
+
+
+@register_block("pre_norm_scaled")
+class ScaledPreNormBlock(Block):
+    """A norm before each sublayer and a weight per channel on its result: x1 = x + s1 * mix(norm1(x)); x2 =
+    x1 + s2 * ffn(norm2(x1)) (without a feed-forward x1); with a `side_input`, x3 = x2 + the normed result of
+    the layer's token input.  A sublayer's result joins the stream in one row kernel (`ops.stream_join`),
+    which writes along what reads the finished rows next: this block's second norm, the stream in the
+    activation dtype for the token input, or the next block's first norm.  A mixture of experts joins by
+    its own last kernel (its `join`)."""
+
+    def __init__(self, spec, dtype, device):
+        from ..config.specs import ConfigError
+        self.dtype = dtype
+        if spec.mixer_norm is None or spec.mixer_scale is None or \
+                (spec.feed_forward is not None and (spec.feed_forward_norm is None or spec.feed_forward_scale is None)):
+            raise ConfigError("a pre_norm_scaled block needs a norm and a scale for every sublayer it has")
+        self.spec = spec
+        self.mixer_norm = make(NORMS, "norm", spec.mixer_norm, dtype, device)
+        self.mixer = make(MIXERS, "mixer", spec.mixer, dtype, device)
+        self.parts = [self.mixer_norm, self.mixer]
+        self.feed_forward = self.side = None
+        if spec.feed_forward is not None:
+            self.feed_forward_norm = make(NORMS, "norm", spec.feed_forward_norm, dtype, device)
+            self.feed_forward = make(FEED_FORWARDS, "feed-forward", spec.feed_forward, dtype, device)
+            self.parts += [self.feed_forward_norm, self.feed_forward]
+        if spec.side_input is not None:
+            self.side = SideInput(spec.side_input, dtype)
+            self.parts.append(self.side)
+        self.s1 = self.s2 = None
+
+    def _scales(self):
+        return [self.spec.mixer_scale] + ([self.spec.feed_forward_scale] if self.feed_forward is not None else [])
+
+    def tensor_requests(self):
+        return [r for p in self.parts for r in p.tensor_requests()] + \
+               [TensorRequest(n, (self.spec.mixer.width,), "norm") for n in self._scales()]
+
+    def bind(self, get):
+        for p in self.parts:
+            p.bind(get)
+        self.s1, self.s2 = ([get(n) for n in self._scales()] + [None])[:2]
+
+    def kv_need(self):
+        return self.mixer.kv_need()
+
+    def state_need(self):
+        return self.mixer.state_need()
+
+    def input_norm(self):
+        return self.mixer_norm
+
+    def first_weights(self, rows):
+        return self.mixer.first_weights(rows)
+
+    def _read(self, norm, x, ctx):
+        h = ctx.take_normed(norm, x)
+        return h if h is not None else norm.forward(x, self.dtype)
+
+    def _along(self, then, x):
+        """What `ops.stream_join` writes beside the stream for the norm (or cast) `then`, or None."""
+        from .norm import StreamCast
+        if isinstance(then, StreamCast):
+            return None if self.dtype == torch.float32 else \
+                (ops.NEXT_COPY, None, None, 0.0, torch.empty(x.shape, dtype=self.dtype, device=x.device))
+        layer, rms = (then.as_layer(), then.as_rms()) if then is not None else (None, None)
+        if layer is None and rms is None:
+            return None
+        normed = torch.empty(x.shape, dtype=self.dtype, device=x.device)
+        return (ops.NEXT_LAYER, *layer, normed) if layer is not None else (ops.NEXT_RMS, rms[0], None, rms[1], normed)
+
+    def _join(self, y, x, weight, ctx, then, norm_eps=None):
+        """x += weight * y (y normed first with `norm_eps`), in place."""
+        along = self._along(then, x)
+        ops.stream_join(y, x, weight, x, norm_eps, along)
+        if along is not None:
+            ctx.keep_normed(then, x, along[4])
+        return x
+
+    def forward(self, x, ctx):
+        after, ctx.after_block_norm, ctx.after_block_weights = ctx.after_block_norm, None, None
+        h = self._read(self.mixer_norm, x, ctx)
+        ctx.next_norm = ctx.next_weights = None           # a row kernel follows every product
+        y = self.mixer.forward(h, ctx)
+        last = self.side.reads if self.side is not None else after
+        if self.feed_forward is None:
+            x = self._join(y, x, self.s1, ctx, last)
+        else:
+            x = self._join(y, x, self.s1, ctx, self.feed_forward_norm)
+            f = self._read(self.feed_forward_norm, x, ctx)
+            ctx.next_norm = ctx.next_weights = None
+            if hasattr(self.feed_forward, "join"):
+                along = self._along(last, x) if self.side is not None else None
+                self.feed_forward.join(f, ctx, x, scale=self.s2, copy=along[4] if along is not None else None)
+                if along is not None:
+                    ctx.keep_normed(last, x, along[4])
+            else:
+                x = self._join(self.feed_forward.forward(f, ctx), x, self.s2, ctx, last)
+        if self.side is None:
+            return x
+        xc = ctx.take_normed(self.side.reads, x)
+        if xc is None:
+            xc = x if self.dtype == torch.float32 else self.side.reads.forward(x, self.dtype)
+        return self._join(self.side.forward(xc, ctx), x, self.side.weight, ctx, after, norm_eps=self.side.eps)

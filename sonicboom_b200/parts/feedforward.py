@@ -167,6 +167,111 @@ class PolyNormFF(FeedForward):
                           residual=residual, act_dtype=self.dtype)
 
 
+@register_feed_forward("relu2")
+class SquaredReluFF(FeedForward):
+    """Feed-forward without a gate whose activation is the square of relu: y = Wdown max(Wup h, 0)^2, no
+    biases.  The up product's epilogue applies the activation; the residual add is fused into the down
+    projection.  `params` may give `names`, the tensor names of the two matrices after the prefix."""
+
+    def __init__(self, spec, dtype, device):
+        self.spec, self.dtype = spec, dtype
+        self.names = tuple(dict(spec.params).get("names", ("up", "down")))
+        self.w_up = self.w_down = None
+
+    def tensor_requests(self):
+        p, d, ff = self.spec.prefix, self.spec.width, self.spec.intermediate
+        return [TensorRequest(p + self.names[0], (ff, d)), TensorRequest(p + self.names[1], (d, ff))]
+
+    def bind(self, get):
+        self.w_up, self.w_down = get(self.spec.prefix + self.names[0]), get(self.spec.prefix + self.names[1])
+
+    def forward(self, h, ctx, residual=None):
+        rows = h.shape[0]
+        t = torch.empty((rows, self.spec.intermediate), dtype=self.dtype, device=h.device)
+        ops.linear(h, self.w_up, t, ops.EPI_RELU2)
+        out = residual if residual is not None else \
+            torch.empty((rows, self.spec.width), dtype=torch.float32, device=h.device)
+        return ctx.linear(t, self.w_down, out,
+                          ops.EPI_RESIDUAL if residual is not None else ops.EPI_NONE,
+                          residual=residual, act_dtype=self.dtype)
+
+
+@register_feed_forward("experts_relu2")
+class ExpertsSquaredRelu(FeedForward):
+    """Mixture of experts over feed-forwards of the form of `relu2`.  Router logits z = R h over `experts` +
+    `identity` outputs in float32; scores s = softmax(z) over all of them; the `top` outputs with the largest
+    s + correction are chosen (the lower index wins a tie) and weighted by s over the chosen ones' sum (+
+    1e-20), times `scale`.  An output from `experts` on is an identity: it hands the input h on.  A shared
+    expert (`shared`, a feed-forward spec, or None) runs for every token and is multiplied by
+    sigmoid(W_sg h), one number per token (`shared_gate`: its tensor name; None: not multiplied).
+    `params`: experts, identity, top, scale, shared, shared_gate, correction (tensor name).  Tensors after
+    the prefix: router [experts + identity, width], the correction [experts + identity], e<j>.up
+    [intermediate, width], e<j>.down [width, intermediate]; the shared gate's [1, width].
+
+    The shared gate's row rides on the router product.  Grouping and tiles are those of
+    `experts_glu_clamped`; the last kernel (`ops.moe_relu2_join`) adds the choices, identities and the gated
+    shared expert and joins the stream, so a block calls `join` rather than `forward`."""
+
+    def __init__(self, spec, dtype, device):
+        from ..config.specs import ConfigError
+        self.spec, self.dtype = spec, dtype
+        p = dict(spec.params)
+        self.n_experts, self.identity, self.top = int(p.get("experts", 0)), int(p.get("identity", 0)), int(p.get("top", 0))
+        self.outputs = self.n_experts + self.identity
+        if self.n_experts < 1 or self.identity < 0 or not 0 < self.top <= self.outputs:
+            raise ConfigError(f"a mixture of {self.n_experts} experts and {self.identity} identities cannot choose {self.top}")
+        self.scale, self.correction_name = float(p.get("scale", 1.0)), p.get("correction", "correction")
+        shared, self.gate_name = p.get("shared"), p.get("shared_gate")
+        self.shared = make(FEED_FORWARDS, "feed-forward", shared, dtype, device) if shared is not None else None
+        if self.shared is None:
+            self.gate_name = None
+        self.w_router = self.correction = self.w_up = self.w_down = None
+
+    def tensor_requests(self):
+        p, d, ff = self.spec.prefix, self.spec.width, self.spec.intermediate
+        req = [TensorRequest(p + "router", (self.outputs, d)), TensorRequest(p + self.correction_name, (self.outputs,), "bias")]
+        for j in range(self.n_experts):
+            req += [TensorRequest(f"{p}e{j}.up", (ff, d)), TensorRequest(f"{p}e{j}.down", (d, ff))]
+        if self.gate_name:
+            req.append(TensorRequest(p + self.gate_name, (1, d)))
+        return req + (self.shared.tensor_requests() if self.shared is not None else [])
+
+    def bind(self, get):
+        p = self.spec.prefix
+        router = [get(p + "router")] + ([get(p + self.gate_name)] if self.gate_name else [])
+        if len({t.dtype for t in router}) > 1:
+            router = [t.float() for t in router]
+        self.w_router = torch.cat(router).contiguous()
+        self.correction = get(p + self.correction_name).float().contiguous()
+        ups = [get(f"{p}e{j}.up") for j in range(self.n_experts)]
+        downs = [get(f"{p}e{j}.down") for j in range(self.n_experts)]
+        if len({t.dtype for t in ups + downs}) > 1:
+            ups, downs = [t.float() for t in ups], [t.float() for t in downs]
+        self.w_up, self.w_down = torch.stack(ups).contiguous(), torch.stack(downs).contiguous()
+        if self.shared is not None:
+            self.shared.bind(get)
+
+    def join(self, h, ctx, x, scale=None, copy=None):
+        """x += scale * (the mixture of h), in place; `copy` receives the finished rows in its dtype."""
+        rows = h.shape[0]
+        ctx.next_norm = ctx.next_weights = None      # the last kernel is not a product: nothing rides on one
+        logits = torch.empty((rows, self.w_router.shape[0]), dtype=torch.float32, device=h.device)
+        ids = torch.empty((rows, self.top), dtype=torch.int32, device=h.device)
+        weights = torch.empty((rows, self.top), dtype=torch.float32, device=h.device)
+        ops.linear(h, self.w_router, logits)
+        ops.moe_route_scored(logits, self.correction, self.top, ids, weights, scale=self.scale, renormalize=True,
+                             scores="softmax")
+        shared = self.shared.forward(h, ctx) if self.shared is not None else None
+        a = h if h.dtype == self.w_up.dtype else ops.cast(h, self.w_up.dtype)
+        return ops.moe_relu2_join(a, ids, weights, self.w_up, self.w_down, x, shared=shared,
+                                  gate=(logits, self.outputs) if self.gate_name else None, scale=scale, copy=copy)
+
+    def forward(self, h, ctx, residual=None):
+        out = residual if residual is not None else \
+            torch.zeros((h.shape[0], self.spec.width), dtype=torch.float32, device=h.device)
+        return self.join(h, ctx, out)
+
+
 @register_feed_forward("experts_glu_clamped")
 class ExpertsClampedGLU(FeedForward):
     """Mixture of experts over clamped gated feed-forwards (the form of `glu_clamped`): router logits

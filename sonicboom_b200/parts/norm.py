@@ -59,24 +59,33 @@ class OnePlusRMSNorm(RMSNorm):
 
 @register_norm("layernorm")
 class LayerNorm(Norm):
-    """Layer norm with a weight and no bias: y = (x - mean) / sqrt(var + eps) * w, the variance
-    being the mean of the squared deviations.  It is not an RMS norm, so no product kernel
-    applies it to its own result (`as_rms` is None) and it runs as a kernel of its own."""
+    """Layer norm with a weight and optionally a bias (the spec names its tensor): y = (x - mean) /
+    sqrt(var + eps) * w [+ b], the variance being the mean of the squared deviations.  It is not an RMS
+    norm, so no product kernel applies it to its own result (`as_rms` is None); `ops.stream_join` writes
+    it along with the rows it finishes, else it runs as a kernel of its own."""
 
     def __init__(self, spec, dtype, device):
-        self.width, self.eps, self.tensor = spec.width, float(spec.eps), spec.tensor
-        self.weight = None
+        self.width, self.eps, self.tensor, self.bias_tensor = spec.width, float(spec.eps), spec.tensor, spec.bias
+        self.weight = self.bias = None
 
     def tensor_requests(self):
-        return [TensorRequest(self.tensor, (self.width,), "norm")]
+        return [TensorRequest(self.tensor, (self.width,), "norm")] + \
+               ([TensorRequest(self.bias_tensor, (self.width,), "bias")] if self.bias_tensor else [])
 
     def bind(self, get):
         self.weight = get(self.tensor)
+        if self.bias_tensor:
+            self.bias = get(self.bias_tensor)
+            if self.bias.dtype != self.weight.dtype:
+                self.weight, self.bias = self.weight.float(), self.bias.float()
+
+    def as_layer(self):
+        return self.weight, self.bias, self.eps
 
     def forward(self, x, out_dtype, rows=None):
         n = x.shape[0] if rows is None else rows.numel()
         out = torch.empty((n, self.width), dtype=out_dtype, device=x.device)
-        return ops.layernorm(x, self.weight, self.eps, out, rows)
+        return ops.layernorm(x, self.weight, self.eps, out, rows, bias=self.bias)
 
 
 class StreamCast(Norm):

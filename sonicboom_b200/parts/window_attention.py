@@ -22,25 +22,58 @@ that attention layers of newer designs combine:
 * `softcap` = c: a score s becomes c tanh(s / c) before the softmax;
 * `gate` = name: a matrix [heads, width]; head h's result is multiplied by the logistic function
   of its product with the mixer's input (it rides on the input product);
+* `conv` = taps: every channel of q, k and v passes a short causal convolution over time right after the
+  projection (tensors: the projection's name + ".conv", [channels, taps]); the last taps - 1 projected
+  values of a sequence are state of the cache;
+* `distance_bias` = (name, most[, rows]): a learned number is added to the capped score, row
+  `distance_bucket(i - j)` of a table [rows, heads] whose rows beyond the first half widen logarithmically
+  up to distance `most` (`rows` is the stored tensor's when not given);
+* `chunk` = n: the query at position i sees key j <= i only when floor(i / n) = floor(j / n), positions
+  counted from the sequence's start; the cache gives the pages of earlier chunks back;
+* `sink` may also be a number: every head's sink has that score;
 * a position encoding with a `magnitude` (stretched rotations) multiplies cosines and sines by it.
 
 Tensors after the prefix: q [heads*head_dim, width], k [kv_heads*head_dim, width], v
 [kv_heads*vdim, width] unless the values are the keys, o [width, heads*vdim], and what the options
 name.  All input projections are one product; `ops.attn_prep` finishes its float32 rows into
-queries and cache rows, the framework's attention kernels run on them unchanged, and
+queries and cache rows (`ops.conv_heads` with a convolution and nothing else to do to the heads), the
+framework's attention kernels run on them unchanged, and
 `ops.attn_unrotate` turns results back and drops the padding where either is needed."""
 from __future__ import annotations
+
+import math
 
 import torch
 
 from .. import ops
-from ..cache.kv import KVNeed
+from ..cache.kv import KVNeed, StateNeed
 from ..weights.loader import TensorRequest
 from .attention import _cat
 from .base import POSITION_ENCODINGS, Mixer, make, register_mixer
 from .rotary import frequency_table
 
 HEAD_STEP = 16          # the tensor-core attention kernels take head sizes in these steps
+
+
+def distance_bucket(n: int, rows: int, most: int) -> int:
+    """The table row for a key n positions back: its own for n below half the rows, then rows that widen
+    logarithmically until distance `most`, then the last."""
+    half = rows // 2
+    if n < half:
+        return n
+    return min(rows - 1, half + math.floor(math.log(n / half) / math.log(most / half) * (rows - half)))
+
+
+def bias_by_distance(table: torch.Tensor, most: int, longest: int = 0) -> torch.Tensor:
+    """float32 [heads, n]: the bias of every distance 0 ... n - 1, the last entry standing for all larger
+    ones (no more than `longest` entries when distances stay below it)."""
+    from ..config.specs import ConfigError
+    rows = table.shape[0]
+    if rows < 2 or 2 * most <= rows:
+        raise ConfigError(f"a distance bias of {rows} rows up to distance {most} (at least 2 rows, half of them below it)")
+    n = most + 1 if longest <= 0 else min(most + 1, longest)
+    index = torch.tensor([distance_bucket(d, rows, most) for d in range(n)], device=table.device)
+    return table.float()[index].t().contiguous()
 
 
 @register_mixer("window_attention")
@@ -57,6 +90,13 @@ class WindowAttention(Mixer):
         self.qk_norm, self.sink_name = p.get("qk_norm"), p.get("sink")
         self.bias_names, self.gate_name = p.get("bias"), p.get("gate")
         self.softcap = float(p.get("softcap", 0.0) or 0.0)
+        self.taps, self.chunk = int(p.get("conv", 0) or 0), int(p.get("chunk", 0) or 0)
+        self.distance_bias = p.get("distance_bias")
+        self.sink_value = None
+        if isinstance(self.sink_name, (int, float)):
+            self.sink_value, self.sink_name = float(self.sink_name), None
+        if self.chunk < 0 or self.taps < 0:
+            raise ConfigError(f"a convolution of {self.taps} taps, chunks of {self.chunk} positions (0: none)")
         head_norm = p.get("head_norm")
         self.head_norm = head_norm[0] if head_norm else None
         if self.head_norm not in (None, "before", "after") or (self.head_norm and self.qk_norm):
@@ -91,10 +131,17 @@ class WindowAttention(Mixer):
         self.gw = self.hq if self.gate_name else 0
         if self.bias_names and self.values_are_keys:
             raise ConfigError("biases of q, k and v need a value projection of its own")
-        self.w_in = self.w_o = self.q_norm = self.k_norm = self.sink = self.b_in = None
+        if self.taps and (self.values_are_keys or self.gate_name):
+            raise ConfigError("a convolution of q, k and v needs a value projection and no gate beside them")
+        # nothing but the convolution happens to a head: its kernel writes queries and cache rows
+        self.conv_only = bool(self.taps) and self.rot == 0 and not self.rotate_values and not self.qk_norm and not self.head_norm
+        self.w_in = self.w_o = self.q_norm = self.k_norm = self.sink = self.b_in = self.w_conv = self.bias = None
 
     def kv_need(self):
-        return KVNeed(self.hkv, self.hd, self.spec.window)
+        return KVNeed(self.hkv, self.hd, self.spec.window, chunk=self.chunk)
+
+    def state_need(self):
+        return StateNeed((self.taps - 1, self.qw + self.kw + self.vw), torch.float32) if self.taps > 1 else None
 
     def tensor_requests(self):
         p, d = self.spec.prefix, self.spec.width
@@ -113,6 +160,11 @@ class WindowAttention(Mixer):
             req.append(TensorRequest(p + self.gate_name, (self.hq, d)))
         if self.sink_name:
             req.append(TensorRequest(p + self.sink_name, (self.hq,), "bias"))
+        if self.taps:
+            req += [TensorRequest(p + n + ".conv", (w, self.taps)) for n, w in ((q, self.qw), (k, self.kw), (v, self.vw))]
+        if self.distance_bias:
+            name, _, rows = (tuple(self.distance_bias) + (None,))[:3]
+            req.append(TensorRequest(p + name, (-1 if rows is None else int(rows), self.hq), "bias"))
         return req
 
     def bind(self, get):
@@ -132,6 +184,12 @@ class WindowAttention(Mixer):
                 self.q_norm, self.k_norm = self.q_norm.float(), self.k_norm.float()
         if self.sink_name:
             self.sink = get(p + self.sink_name).float().contiguous()
+        elif self.sink_value is not None:
+            self.sink = torch.full((self.hq,), self.sink_value, dtype=torch.float32, device=self.w_o.device)
+        if self.taps:
+            self.w_conv = _cat([get(p + n + ".conv") for n in (q, k, v)])
+        if self.distance_bias:
+            self.bias = bias_by_distance(get(p + self.distance_bias[0]), int(self.distance_bias[1]), self.chunk)
 
     def first_weights(self, rows):
         n, k = self.w_in.shape
@@ -150,14 +208,26 @@ class WindowAttention(Mixer):
         else:
             ops.linear(h, self.w_in[:width_in], proj)
         q = torch.empty((rows, self.hq, self.hd), dtype=self.dtype, device=h.device)
-        ops.attn_prep(proj, 0, k_off, -1 if self.values_are_keys else k_off + self.kw, self.hq, self.hkv,
-                      self.dim, self.vdim, self.hd, self.rot, self.interleaved, self.inv_freq, self.v_inv_freq,
-                      self.q_norm, self.k_norm, self.eps, plan.row_seq, plan.row_pos, g.page_off, g.page_ids,
-                      g.page_size, storage if ctx.owns_cache else None, q, head_norm=self.head_norm,
-                      rot_scale=self.rot_scale)
+        if self.taps and not ctx.owns_cache:
+            from ..config.specs import ConfigError
+            raise ConfigError("attention with convolved projections has keys and values of its own")
+        state = ctx.state() if self.taps > 1 else None
+        if self.conv_only and self.taps <= ops.conv_heads_max_taps():
+            ops.conv_heads(proj, self.w_conv, plan, g.page_off, g.page_ids, g.page_size, self.hq, self.hkv, self.dim,
+                           self.vdim, state, storage, q)
+        else:
+            if self.taps:
+                turned = torch.empty_like(proj)
+                proj = ops.causal_conv(proj, 0, width_in, self.w_conv, None, plan, state, turned)
+            ops.attn_prep(proj, 0, k_off, -1 if self.values_are_keys else k_off + self.kw, self.hq, self.hkv,
+                          self.dim, self.vdim, self.hd, self.rot, self.interleaved, self.inv_freq, self.v_inv_freq,
+                          self.q_norm, self.k_norm, self.eps, plan.row_seq, plan.row_pos, g.page_off, g.page_ids,
+                          g.page_size, storage if ctx.owns_cache else None, q, head_norm=self.head_norm,
+                          rot_scale=self.rot_scale)
         mixed = torch.empty((rows, self.hq * self.hd), dtype=self.dtype, device=h.device)
         ops.attention(q, mixed, plan, ctx.kv_group(), storage, self.hq, self.hkv, self.hd, self.spec.window,
-                      self.spec.scale, warm=self.w_o, sink=self.sink, softcap=self.softcap)
+                      self.spec.scale, warm=self.w_o, sink=self.sink, softcap=self.softcap, chunk=self.chunk,
+                      bias=self.bias)
         if self.rotate_values or self.hd != self.vdim or self.gw:
             turned = torch.empty((rows, self.hq * self.vdim), dtype=self.dtype, device=h.device)
             mixed = ops.attn_unrotate(mixed, turned, self.hq, self.hd, self.vdim, self.interleaved,
