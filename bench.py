@@ -7,6 +7,7 @@ sizes of Qwen2.5-7B with random weights on one B200.
     python bench.py --arch mefupel [--sizes w2048,w3584] [--prompt 2048] [--batch 8] [--steps K]
     python bench.py --arch leguvik [--sizes w2048,w3584] [--prompt 2048] [--batch 8] [--steps K]
     python bench.py --arch bulodra [--sizes w2048,w3584] [--prompt 2048] [--batch 8] [--steps K]
+    python bench.py --arch debisun [--sizes w2048,w3584] [--prompt 2048] [--batch 8] [--steps K]
 
 Prints ONE JSON line.  (`--arch zolulix` is a measurement of its own: the Zolulix design beside the
 Qwen2.5 decoder of equal sizes and its kernels alone; without it the workload below runs.)  A "step" is one decode step of the whole batch.  The default run is a
@@ -1191,6 +1192,216 @@ def run_bulodra(args) -> int:
     return 0
 
 
+# ---------------------------------------------------------------------------- --arch debisun
+def debisun_config(width, n_layers, vocab, heads, kv_heads, dim, chunk, taps, bias_rows, bias_max, side, experts,
+                   identity, top, expert_ff, shared_ff, dense_ff):
+    """A Debisun model of the given layer sizes: the first layer with a dense feed-forward, the others
+    with a mixture of experts, identities and a shared expert."""
+    mixer = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "softcap": 40.0,
+             "conv": taps, "bias_rows": bias_rows, "bias_max": bias_max, "mask": {"size": chunk}}
+    moe = {"kind": "moe", "router": {"experts": experts, "identity": identity, "top": top, "scale": 2.0},
+           "expert": {"ff": expert_ff}, "shared": {"ff": shared_ff}}
+    layers = [{"type": "attention", "mixer": mixer, "mlp": {"kind": "dense", "ff": dense_ff} if i == 0 else moe}
+              for i in range(n_layers)]
+    return {"architecture": "Debisun", "vocab": vocab, "width": width, "norm": {"eps": 1e-5},
+            "token_side": {"dim": side}, "layers": layers}
+
+
+def debisun_bulodra_config(z):
+    """The Bulodra model beside it: every layer with capped attention in a window as long as the chunk, the
+    same width, depth, vocabulary, heads, experts, choices and expert sizes."""
+    b = bulodra_config(width=z["width"], n_layers=1, vocab=z["vocab"], heads=z["heads"], kv_heads=z["kv_heads"], dim=z["dim"],
+                       window=z["chunk"], l_dim=64, l_rot=32, l_vdim=64, kv_rank=96, q_rank=512, experts=z["experts"],
+                       top=z["top"], groups=(4, 2), expert_ff=z["expert_ff"], shared_ff=z["shared_ff"], dense_ff=z["dense_ff"])
+    mixer = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["dim"], "scale": z["dim"] ** -0.5,
+             "softcap": 40.0, "mask": {"size": z["chunk"]}, "rot": {"base": 1e4, "dims": z["dim"] // 2}}
+    moe = {"kind": "moe", "router": {"experts": z["experts"], "top": z["top"], "scale": 2.0, "groups": {"count": 4, "keep": 2}},
+           "expert": {"ff": z["expert_ff"], "limit": 7.0}, "shared": {"ff": z["shared_ff"], "limit": 7.0}}
+    b["layers"] = [{"type": "attention_2", "mixer": mixer, "mlp": {"kind": "dense", "ff": z["dense_ff"]} if i == 0 else moe}
+                   for i in range(z["n_layers"])]
+    return b
+
+
+DEBISUN_SIZES = {
+    # Bulodra is the closest design (capped softmax attention of a bounded reach, a mixture of experts chosen by
+    # scores with a correction, a shared expert); its gated feed-forwards have a third matrix
+    "w2048": dict(width=2048, n_layers=8, vocab=32768, heads=16, kv_heads=4, dim=128, chunk=1536, taps=4, bias_rows=32,
+                  bias_max=128, side=256, experts=32, identity=8, top=4, expert_ff=1024, shared_ff=2048, dense_ff=8192),
+    "w3584": dict(width=3584, n_layers=8, vocab=32768, heads=28, kv_heads=4, dim=128, chunk=8192, taps=4, bias_rows=64,
+                  bias_max=4096, side=256, experts=64, identity=16, top=6, expert_ff=1536, shared_ff=3072, dense_ff=18944),
+}
+
+
+def debisun_kernels(bench, z, rows, context):
+    """Each kernel that came with Debisun (or was extended for it) alone at `rows` rows (one sequence
+    of `rows` tokens when rows > 64, else `rows` sequences that hold `context` tokens each and go on
+    by one), with the bytes it must read and write once, and beside each the like kernel of the
+    framework's other models at the same sizes."""
+    import torch
+    from sonicboom_b200 import ops
+    from sonicboom_b200.cache.kv import Cache, KVNeed, StateNeed
+    from sonicboom_b200.engine.step import StepEntry, StepPlan
+    from sonicboom_b200.parts.rotary import frequency_table
+    from sonicboom_b200.parts.window_attention import bias_by_distance
+    dev, pk, timed = bench.dev, bench.pk, bench.timed
+    W, bf = z["width"], torch.bfloat16
+    out = {}
+
+    def rec(name, ms, nbytes, flops=0):
+        out[name] = {"us": round(ms * 1e3, 2), "bytes": int(nbytes),
+                     "hbm_frac": round(nbytes / (ms / 1e3) / 1e9 / pk["hbm_gbs"], 3)}
+        if flops:
+            out[name]["tflops"] = round(flops / (ms / 1e3) / 1e12, 2)
+    prompt = rows > 64
+    n_seqs, new = (1, rows) if prompt else (rows, 1)
+    past = 0 if prompt else context
+    H, G, d, chunk, taps = z["heads"], z["kv_heads"], z["dim"], z["chunk"], z["taps"]
+    channels = (H + 2 * G) * d
+    reach = past % chunk + 1                            # keys a decoded token sees within its chunk
+    cache = Cache([KVNeed(G, d)], [StateNeed((taps - 1, channels), torch.float32)], n_seqs * (past + new + 64), bf, dev,
+                  n_slots=n_seqs)
+    slots = [cache.open() for _ in range(n_seqs)]
+    for s in slots:
+        if past:
+            cache.reserve(s, past)
+            cache.advance(s, past)
+        cache.reserve(s, past + new)
+    plan = StepPlan(cache, [StepEntry(s, [0] * new, []) for s in slots], dev)
+    kind = f"{n_seqs} sequence(s) of {new}" + (f" after {past}" if past else "")
+    g0, store = plan.groups[0], cache.groups[0].entry_storage(0)
+    store.normal_()
+    # rows of the stream
+    x, y = torch.randn(rows, W, device=dev), torch.randn(rows, W, device=dev)
+    wb = torch.ones(W, device=dev, dtype=bf)
+    xo, nb = torch.empty(rows, W, device=dev), torch.empty(rows, W, device=dev, dtype=bf)
+    rec("stream_join + layer norm", timed(lambda: ops.stream_join(y, x, wb, xo, None, (ops.NEXT_LAYER, wb, wb, 1e-5, nb))), rows * W * 14)
+    rec("stream_join, result normed, + layer norm",
+        timed(lambda: ops.stream_join(y, x, wb, xo, 1e-5, (ops.NEXT_LAYER, wb, wb, 1e-5, nb))), rows * W * 14)
+    rec("like: norm_add + next norm", timed(lambda: ops.norm_add(y, x, wb, 1e-6, xo, (wb, 1e-6, nb))), rows * W * 14)
+    rec("layernorm with a bias", timed(lambda: ops.layernorm(x, wb, 1e-5, nb, bias=wb)), rows * W * 6)
+    rec("like: layernorm", timed(lambda: ops.layernorm(x, wb, 1e-5, nb)), rows * W * 6)
+    # queries and cache rows
+    proj = torch.randn(rows, channels, device=dev)
+    wc = torch.randn(channels, taps, device=dev).to(bf)
+    q = torch.randn(rows, H, d, device=dev).to(bf)
+    state_bytes = n_seqs * (taps - 1) * channels * 8
+    rec("conv_heads", timed(lambda: ops.conv_heads(proj, wc, plan, g0.page_off, g0.page_ids, g0.page_size, H, G, d, d,
+                                                   cache.state[0], store, q)), rows * channels * 6 + state_bytes)
+    table = frequency_table(1e4, d, dev)
+    rec("like: attn_prep, every head normed after the rotation",
+        timed(lambda: ops.attn_prep(proj, 0, H * d, (H + G) * d, H, G, d, d, d, d // 2, False, table, None, None, None, 1e-6,
+                                    plan.row_seq, plan.row_pos, g0.page_off, g0.page_ids, g0.page_size, store, q,
+                                    head_norm="after")), rows * channels * 6)
+    turned = torch.empty(rows, channels, device=dev)
+    rec("like: causal_conv", timed(lambda: ops.causal_conv(proj, 0, channels, wc, None, plan, cache.state[0], turned)),
+        rows * channels * 8 + state_bytes)
+    # attention
+    q.normal_()
+    o = torch.empty(rows, H * d, device=dev, dtype=bf)
+    bias = ops.DistanceBias(bias_by_distance(torch.randn(z["bias_rows"], H), z["bias_max"], chunk).to(dev))
+    sink = torch.zeros(H, device=dev)
+    if prompt:
+        c_keys, w_keys = sum(i % chunk + 1 for i in range(rows)), sum(min(i + 1, chunk) for i in range(rows))
+        c_bytes = w_bytes = rows * G * d * 4
+    else:
+        c_keys, w_keys = rows * reach, rows * min(past + 1, reach)
+        c_bytes, w_bytes = c_keys * G * d * 4, w_keys * G * d * 4
+    scale = d ** -0.5
+
+    def att(win, **kw):
+        return timed(lambda: ops.attention(q, o, plan, 0, store, H, G, d, win, scale, **kw))
+    rec(f"attention, chunks of {chunk}, capped scores, distance bias, sink ({kind})",
+        att(0, softcap=40.0, chunk=chunk, bias=bias, sink=sink), c_bytes + rows * H * d * 4 + bias.values.numel() * 4, 4 * c_keys * H * d)
+    rec(f"attention, chunks of {chunk}, capped scores ({kind})", att(0, softcap=40.0, chunk=chunk),
+        c_bytes + rows * H * d * 4, 4 * c_keys * H * d)
+    win = chunk if prompt else reach                    # a window of as many keys
+    rec(f"like: attention, capped scores ({kind}; window {win})", att(win, softcap=40.0), w_bytes + rows * H * d * 4, 4 * w_keys * H * d)
+    rec(f"like: attention ({kind}; window {win})", att(win), w_bytes + rows * H * d * 4, 4 * w_keys * H * d)
+    # the router and the experts
+    E, I, top, ff = z["experts"], z["identity"], z["top"], z["expert_ff"]
+    logits = torch.randn(rows, E + I + 1, generator=bench.gen).to(dev)
+    corr = torch.zeros(E + I, device=dev)
+    ids, wts = torch.empty(rows, top, dtype=torch.int32, device=dev), torch.empty(rows, top, device=dev)
+    rec("moe_route_scored, softmax", timed(lambda: ops.moe_route_scored(logits, corr, top, ids, wts, scale=2.0, renormalize=True,
+                                                                        scores="softmax")), rows * ((E + I) * 4 + top * 8))
+    slog, scorr = logits[:, :E].contiguous(), corr[:E].contiguous()
+    rec("like: moe_route_scored (groups)", timed(lambda: ops.moe_route_scored(slog, scorr, top, ids, wts, groups=(4, 2), scale=2.0)),
+        rows * (E * 4 + top * 8))
+    h = torch.randn(rows, W, device=dev).to(bf)
+    w1 = torch.randn(E, ff, W, device=dev, dtype=bf) * 0.02
+    w2 = torch.randn(E, W, ff, device=dev, dtype=bf) * 0.02
+    w1g = torch.randn(E, 2, ff, W, device=dev, dtype=bf) * 0.02
+    hit = len(set(ids.flatten().tolist()))              # experts that some token chose (ids without identities here)
+    pairs = rows * top
+    pair_io = pairs * ff * 4 + pairs * W * 4
+    rec("experts: group, up with squared relu, down", timed(lambda: ops._moe_pairs(h, ids, w1, w2, ops.EXPERT_RELU2, 0.0, 0.0)),
+        hit * 2 * ff * W * 2 + rows * W * 2 + pair_io, 4 * pairs * ff * W)
+    rec("like: experts: group, gated up, down", timed(lambda: ops._moe_pairs(h, ids, w1g, w2, ops.EXPERT_CLAMPED, 7.0, 1.7)),
+        hit * 3 * ff * W * 2 + rows * W * 2 + pair_io, 6 * pairs * ff * W)
+    from sonicboom_b200.ops import _check, _code, _ptr, _stream, lib
+    pair_out = torch.randn(pairs, W, device=dev)
+    rec("moe_join: choices, identities, gated shared expert, scale, copy", timed(lambda: _check(lib().sb_moe_join(
+        _ptr(x), _ptr(pair_out), _ptr(ids), _ptr(wts), E, _ptr(h), _code(bf), _ptr(y), _ptr(logits), E + I + 1, _ptr(wb), _code(bf),
+        rows, top, W, _ptr(nb), _code(bf), _stream()), "moe_join")), pairs * W * 4 + rows * W * 16)
+    rec("like: moe_combine", timed(lambda: _check(lib().sb_moe_combine(_ptr(x), _ptr(pair_out), _ptr(wts), rows, top, W, _stream()),
+                                                  "moe_combine")), pairs * W * 4 + rows * W * 8)
+    # the dense feed-forward's first product, at as many weight rows
+    dff = z["dense_ff"]
+    wu = torch.randn(2 * dff, W, device=dev, dtype=bf) * 0.02
+    a2, a1 = torch.empty(rows, 2 * dff, device=dev, dtype=bf), torch.empty(rows, dff, device=dev, dtype=bf)
+    rec("product with squared relu in its epilogue", timed(lambda: ops.linear(h, wu, a2, ops.EPI_RELU2)),
+        2 * dff * W * 2 + rows * (W + 2 * dff) * 2, 4 * rows * dff * W)
+    rec("like: gate | up product with gelu in its epilogue", timed(lambda: ops.linear(h, wu, a1, ops.EPI_SWIGLU, gate_kind=ops.GATE_GELU_TANH)),
+        2 * dff * W * 2 + rows * (W + dff) * 2, 4 * rows * dff * W)
+    # the token input
+    sd = z["side"]
+    wg, wp = torch.randn(sd, W, device=dev, dtype=bf) * 0.02, torch.randn(W, sd, device=dev, dtype=bf) * 0.02
+    zz, gg = torch.randn(rows, sd, device=dev), torch.randn(rows, sd, device=dev).to(bf)
+    tab = torch.randn(z["vocab"], 4 * sd, device=dev, dtype=bf)
+    toks = torch.randint(0, z["vocab"], (rows,), generator=bench.gen).int().to(dev)
+    rec("token input: gate product", timed(lambda: ops.linear(h, wg, zz)), sd * W * 2 + rows * (W * 2 + sd * 4), 2 * rows * sd * W)
+    rec("token input: side_gate", timed(lambda: ops.side_gate(zz, toks, tab, sd, gg)), rows * sd * 8)
+    gu = torch.randn(rows, 2 * sd, device=dev)
+    rec("like: gated_act", timed(lambda: ops.gated_act(gu, ops.GATE_GELU_TANH, gg)), rows * sd * 10)
+    rec("token input: product back", timed(lambda: ops.linear(gg, wp, xo)), sd * W * 2 + rows * (W * 4 + sd * 2), 2 * rows * sd * W)
+    return out
+
+
+def run_debisun(args) -> int:
+    """Prefill and decode throughput of Debisun models at layer sizes of real models (random
+    weights) beside the Bulodra models of equal width, depth, vocabulary, attention and experts; and
+    each of its kernels alone beside the like kernels of the other models."""
+    import torch
+    import sonicboom_b200 as sb
+    from sonicboom_b200 import ops
+
+    bench = ArchBench()
+    dev = bench.dev
+    result = {"arch": "debisun", "impl": "ours", "dtype": "bf16", "peaks": bench.pk, "sizes": {},
+              "data": "synthetic: random N(0,0.02) weights, uniform random token ids",
+              "timing": "CUDA events; kernels alone: median of 5 after 3 warm-up calls, L2 flushed "
+                        "(256 MB written) before each; models: prefill median of 3, decode one region of K steps"}
+    with ClockSampler() as clocks:
+        for name, z in DEBISUN_SIZES.items():
+            if args.sizes and name not in args.sizes.split(","):
+                continue
+            rec = {"debisun_config": dict(z)}
+            for label, cfg in (("debisun", debisun_config(**z)),
+                               ("bulodra (equal width, depth, vocab, heads, experts; window as long as the chunk)",
+                                debisun_bulodra_config(z))):
+                m = sb.random_model(cfg, seed=0, dtype="bfloat16", device=dev, std=0.02)
+                rec[label] = bench.model_points(m, args.prompt, args.batch, args.steps, args.warmup)
+                del m
+                torch.cuda.empty_cache()
+            for rows in (args.prompt, args.batch):
+                rec["kernels_rows_%d" % rows] = debisun_kernels(bench, z, rows, args.prompt)
+            result["sizes"][name] = rec
+    ops.check_status()
+    result["clocks"] = clocks.summary()
+    print(json.dumps(result))
+    return 0
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1210,15 +1421,15 @@ def main() -> int:
                     help="run one phase only and print a short line (small cases for profilers)")
     ap.add_argument("--eager", action="store_true",
                     help="with --only decode: launch the step kernel by kernel, not as a graph")
-    ap.add_argument("--arch", choices=["qwen2", "zolulix", "mefupel", "leguvik", "bulodra"], default="qwen2",
+    ap.add_argument("--arch", choices=["qwen2", "zolulix", "mefupel", "leguvik", "bulodra", "debisun"], default="qwen2",
                     help="zolulix: that design's prefill and decode throughput and its kernels alone, "
                          "beside the Qwen2.5 decoder of equal sizes (its own JSON line; the default "
                          "workload is unchanged); mefupel: the same for that design, beside Zolulix and "
                          "Qwen2.5 models of equal sizes; leguvik: the same for that design, beside Mefupel "
                          "models of equal sizes; bulodra: the same for that design, beside Leguvik models of "
-                         "equal sizes")
-    ap.add_argument("--sizes", default="", help="with --arch zolulix / mefupel / leguvik / bulodra: which of its sizes to run (comma separated)")
-    ap.add_argument("--prompt", type=int, default=2048, help="with --arch zolulix / mefupel / leguvik / bulodra: prompt length")
+                         "equal sizes; debisun: the same for that design, beside Bulodra models of equal sizes")
+    ap.add_argument("--sizes", default="", help="with --arch zolulix / mefupel / leguvik / bulodra / debisun: which of its sizes to run (comma separated)")
+    ap.add_argument("--prompt", type=int, default=2048, help="with --arch zolulix / mefupel / leguvik / bulodra / debisun: prompt length")
     args = ap.parse_args()
     if args.impl == "reference":
         return reference_arm()
@@ -1235,6 +1446,8 @@ def main() -> int:
         return run_leguvik(args)
     if args.arch == "bulodra":
         return run_bulodra(args)
+    if args.arch == "debisun":
+        return run_debisun(args)
     return run(args)
 
 

@@ -111,6 +111,8 @@ __device__ __forceinline__ void dt_tile_step(uint32_t qs, uint32_t ks, uint32_t 
     }
   }
   const int t = lane & 3;
+  const float* ba = BIAS ? bias_of(ra, key0, 32, bias_last) + (31 - 2 * t) : nullptr;
+  const float* bb = BIAS ? bias_of(rb, key0, 32, bias_last) + (31 - 2 * t) : nullptr;
   float tmax[2] = {-INFINITY, -INFINITY};
 #pragma unroll
   for (int j = 0; j < 4; ++j) {
@@ -119,7 +121,8 @@ __device__ __forceinline__ void dt_tile_step(uint32_t qs, uint32_t ks, uint32_t 
       const int key = key0 + j * 8 + 2 * t + (i & 1);
       const RowView& rv = (i < 2) ? ra : rb;
       const bool seen = key <= rv.pos && key >= rv.lo;
-      const float v = seen ? row_score<BIAS>(s[j][i], sm, rv, key, bias_last) : -INFINITY;
+      const float score = BIAS ? biased_score(s[j][i], sm, __ldg((i < 2 ? ba : bb) - (j * 8 + (i & 1)))) : mapped_score(s[j][i], sm);
+      const float v = seen ? score : -INFINITY;
       s[j][i] = v;
       tmax[i >> 1] = fmaxf(tmax[i >> 1], v);
     }

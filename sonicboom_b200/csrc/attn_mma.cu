@@ -26,9 +26,11 @@
 // i - j < window) (core/src/nn/attention.cpp:66-70); with a chunk size c > 0 also only when j lies
 // in the query's own chunk, floor(j / c) = floor(i / c).  Both are a lowest visible key that grows
 // with i (low_key).  The scale multiplies the finished dot product in float32.  With a distance
-// bias (`bias` [n_q_heads][bias_len]) the finished, capped score gets bias[h][min(i - j, bias_len - 1)]
-// added; the kernels that do so are instantiations of their own (BIAS), so that others carry
-// nothing of it.  Probabilities are rounded to bfloat16 only as the P.V operand.
+// bias the finished, capped score gets b_h(min(i - j, bias_len - 1)) added; the kernels that do so are
+// instantiations of their own (BIAS), so that others carry nothing of it.  Its table holds log2(e) b_h, a
+// row of BIAS_PAD + bias_len + BIAS_PAD values a head: zeros for negative distances, the biases, the last
+// one repeated.  So a tile of at most BIAS_PAD keys reads one stretch of a row, whose start is clamped
+// once, at fixed offsets.  Probabilities are rounded to bfloat16 only as the P.V operand.
 #include <math.h>
 
 #include "common.cuh"
@@ -54,6 +56,7 @@ constexpr int SPLIT_PAGES = 4, LONG_SPLIT_PAGES = 8, LONG_LEN = 4096;
 __host__ __device__ constexpr int split_pages_for(int len) { return len > LONG_LEN ? LONG_SPLIT_PAGES : SPLIT_PAGES; }
 constexpr int DEC_ROWS = 16;
 constexpr float LOG2E = 1.4426950408889634f;
+constexpr int BIAS_PAD = 64;
 
 static_assert(HD % 16 == 0 && HD >= 16 && HD <= 256, "head size in steps of 16, at most 256");
 
@@ -72,7 +75,7 @@ struct AttnParams {
   int n_seqs;
   float scale_log2;            // scale * log2(e)
   float cap_a, cap_b;          // a score cap c > 0: cap_a = scale / c, cap_b = c log2(e); else both 0
-  const float* bias;           // [n_q_heads][bias_len] by distance, the last one for all larger ones (or null)
+  const float* bias;           // [n_q_heads][BIAS_PAD + bias_len + BIAS_PAD] by distance (or null)
   int bias_len;
   const float* sink;           // [n_q_heads] or null: exp(sink) joins each row's softmax denominator
   const char* warm;            // decode: bytes the next kernel will read, asked into L2 (or null)
@@ -105,20 +108,22 @@ __device__ __forceinline__ int low_key(const AttnParams& p, int pos) {
   return p.chunk > 0 ? max(w, pos / p.chunk * p.chunk) : w;
 }
 // What a thread needs to know of one of its query rows: the row's position (-1: a padding row, which
-// sees nothing), its first visible key, and its head's row of the distance bias.
+// sees nothing), its first visible key, and its head's distance bias (at distance 0).
 struct RowView {
   int pos, lo;
   const float* bias;
 };
 template <bool BIAS>
 __device__ __forceinline__ RowView row_view(const AttnParams& p, int pos, int head) {
-  return RowView{pos, low_key(p, max(pos, 0)), BIAS ? p.bias + (size_t)head * p.bias_len : nullptr};
+  return RowView{pos, low_key(p, max(pos, 0)), BIAS ? p.bias + (size_t)head * (p.bias_len + 2 * BIAS_PAD) + BIAS_PAD : nullptr};
 }
-// The exponent's argument of one visible key's score, with the row's distance bias.
-template <bool BIAS>
-__device__ __forceinline__ float row_score(float dot, const ScoreMap& sm, const RowView& rv, int key, int bias_last) {
-  const float v = mapped_score(dot, sm);
-  return BIAS ? fmaf(__ldg(rv.bias + min(max(rv.pos - key, 0), bias_last)), LOG2E, v) : v;
+// The biases of n <= BIAS_PAD keys from key0 on: the key key0 + i reads element n - 1 - i.
+__device__ __forceinline__ const float* bias_of(const RowView& rv, int key0, int n, int bias_last) {
+  return rv.bias + min(max(rv.pos - key0 - (n - 1), -BIAS_PAD), bias_last);
+}
+// The exponent's argument of one key's score plus its (scaled) bias.
+__device__ __forceinline__ float biased_score(float dot, const ScoreMap& sm, float b) {
+  return sm.cap_b != 0.0f ? fmaf(sm.cap_b, tanh_approx(dot * sm.cap_a), b) : fmaf(dot, sm.scale_log2, b);
 }
 
 __device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0,
@@ -193,6 +198,8 @@ __device__ __forceinline__ void tile_step(const uint32_t (&qf)[HD / 16][4], uint
     }
   }
   const int t = lane & 3;
+  const float* ba = BIAS ? bias_of(ra, key0, NKEYS, bias_last) + (NKEYS - 1 - 2 * t) : nullptr;
+  const float* bb = BIAS ? bias_of(rb, key0, NKEYS, bias_last) + (NKEYS - 1 - 2 * t) : nullptr;
   float tmax[2] = {-INFINITY, -INFINITY};
 #pragma unroll
   for (int j = 0; j < NKEYS / 8; ++j) {
@@ -201,7 +208,8 @@ __device__ __forceinline__ void tile_step(const uint32_t (&qf)[HD / 16][4], uint
       const int key = key0 + j * 8 + 2 * t + (i & 1);
       const RowView& rv = (i < 2) ? ra : rb;
       const bool seen = key <= rv.pos && key >= rv.lo;
-      const float v = seen ? row_score<BIAS>(s[j][i], sm, rv, key, bias_last) : -INFINITY;
+      const float score = BIAS ? biased_score(s[j][i], sm, __ldg((i < 2 ? ba : bb) - (j * 8 + (i & 1)))) : mapped_score(s[j][i], sm);
+      const float v = seen ? score : -INFINITY;
       s[j][i] = v;
       tmax[i >> 1] = fmaxf(tmax[i >> 1], v);
     }

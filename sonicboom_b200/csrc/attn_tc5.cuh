@@ -334,10 +334,28 @@ attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_kv, const AttnPa
       // every key of the page visible to every row of the tile: no mask to apply
       const bool open = key0 + KT - 1 <= p_lo && key0 >= lo_hi;
       if (BIAS) {
-        // a bias is not monotone in the dot product: finished scores from here on
+        // A bias is not monotone in the dot product: finished scores from here on.  Far from the diagonal
+        // every key of the page has the table's last bias, and nothing is read.
+        const float* brow = bias_of(rv, key0, KT, bias_last);
+        if (__all_sync(0xffffffffu, rv.pos < 0 || rv.pos - key0 - (KT - 1) >= bias_last)) {
+          const float b = rv.bias[bias_last];
+          if (capped) {
 #pragma unroll
-        for (int i = 0; i < KT; ++i)
-          sv[i] = __float_as_uint(row_score<true>(__uint_as_float(sv[i]), sm, rv, key0 + i, bias_last));
+            for (int i = 0; i < KT; ++i)
+              sv[i] = __float_as_uint(fmaf(sm.cap_b, tanh_approx(__uint_as_float(sv[i]) * sm.cap_a), b));
+          } else {
+#pragma unroll
+            for (int i = 0; i < KT; ++i) sv[i] = __float_as_uint(fmaf(__uint_as_float(sv[i]), sm.scale_log2, b));
+          }
+        } else if (capped) {
+#pragma unroll
+          for (int i = 0; i < KT; ++i)
+            sv[i] = __float_as_uint(fmaf(sm.cap_b, tanh_approx(__uint_as_float(sv[i]) * sm.cap_a), __ldg(brow + (KT - 1 - i))));
+        } else {
+#pragma unroll
+          for (int i = 0; i < KT; ++i)
+            sv[i] = __float_as_uint(fmaf(__uint_as_float(sv[i]), sm.scale_log2, __ldg(brow + (KT - 1 - i))));
+        }
       }
       if (!open) {
 #pragma unroll

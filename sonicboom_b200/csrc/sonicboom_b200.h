@@ -426,7 +426,8 @@ int sb_attention_last_launches(void);     /* kernels the last sb_attention call 
 size_t sb_attention_scratch_bytes(int n_rows, int n_q_heads, int n_kv_heads, int max_new,
                                   int max_len);
 /* Causal grouped-query attention of a step's rows over one cache entry's pages (bfloat16).
- * sink, chunk, bias: as in sb_attention_plain. */
+ * sink, chunk: as in sb_attention_plain.  bias: null, or float32 [n_q_heads][64 + bias_len + 64], the biases of
+ * sb_attention_plain times log2(e) with 64 zeros before them and the last one 64 times more after them. */
 int sb_attention(const void* q, void* out, int n_rows, int n_seqs, int max_new,
                  const int32_t* seq_row0, const int32_t* seq_pos0, const int32_t* page_off,
                  const int32_t* page_ids, int page_size, const void* cache, int n_q_heads,

@@ -499,17 +499,33 @@ def attention_lib(head_dim: int):
     return _attn_libs[head_dim]
 
 
+BIAS_PAD = 64                    # keys of a tile of the tensor-core attention kernels: values around their bias table
+
+
+class DistanceBias:
+    """A number per query head and distance that joins an attention score: `values` float32 [heads, n] for the
+    distances 0 ... n - 1, the last one standing for all larger distances.  `padded` is the table as the
+    tensor-core kernels read it: times log2(e), zeros in front, the last value repeated behind."""
+
+    def __init__(self, values: torch.Tensor):
+        assert values.dtype == torch.float32 and values.dim() == 2 and values.shape[1] >= 1
+        self.values = values.contiguous()
+        scaled = self.values * 1.4426950408889634
+        zeros = torch.zeros((values.shape[0], BIAS_PAD), dtype=torch.float32, device=values.device)
+        self.padded = torch.cat([zeros, scaled, scaled[:, -1:].expand(-1, BIAS_PAD)], dim=1).contiguous()
+
+
 def attention(q: torch.Tensor, out: torch.Tensor, plan, group_index: int, cache: torch.Tensor,
               n_q_heads: int, n_kv_heads: int, head_dim: int, window: int, scale: float,
               kernel: str = "auto", warm: torch.Tensor | None = None,
               sink: torch.Tensor | None = None, softcap: float = 0.0, chunk: int = 0,
-              bias: torch.Tensor | None = None) -> torch.Tensor:
+              bias: DistanceBias | None = None) -> torch.Tensor:
     """Causal grouped-query attention of the step's rows over one cache entry's pages.
     `sink` (float32, one per query head): exp(sink) joins that head's softmax denominator.
     `softcap` c > 0: a score s becomes c tanh(s / c) before the softmax.
     `chunk` c > 0: only keys of the query's own stretch of c positions, counted from the sequence's
-    start, are visible.  `bias` (float32 [query heads, n]): the capped score of a key d positions back
-    gets bias[h, min(d, n - 1)] added.
+    start, are visible.  `bias`: the capped score of a key d positions back gets the head's bias for
+    distance d added (`DistanceBias`).
 
     bfloat16 runs the tensor-core kernels (built for the head size at first use); float32, a
     head size those kernels do not take, or `kernel="plain"` run the plain kernel.  `"mma"` keeps
@@ -523,8 +539,8 @@ def attention(q: torch.Tensor, out: torch.Tensor, plan, group_index: int, cache:
     if sink is not None:
         assert sink.dtype == torch.float32 and sink.numel() == n_q_heads
     if bias is not None:
-        assert bias.dtype == torch.float32 and bias.dim() == 2 and bias.shape[0] == n_q_heads
-    bias_len = bias.shape[1] if bias is not None else 0
+        assert bias.values.shape[0] == n_q_heads
+    bias_len = bias.values.shape[1] if bias is not None else 0
     al = attention_lib(head_dim) if (q.dtype == torch.bfloat16 and cache.dtype == torch.bfloat16
                                      and kernel != "plain") else None
     if al is not None:
@@ -540,7 +556,8 @@ def attention(q: torch.Tensor, out: torch.Tensor, plan, group_index: int, cache:
             head_dim, window, ctypes.c_float(scale), _ptr(scratch),
             ctypes.c_size_t(scratch.numel() if scratch is not None else 0),
             _ptr(counters), counters.numel(), plan.max_len, cache.shape[0], _sm_count(q.device),
-            *_warm_args(warm), _ptr(sink), ctypes.c_float(softcap), int(chunk), _ptr(bias), bias_len, _stream())
+            *_warm_args(warm), _ptr(sink), ctypes.c_float(softcap), int(chunk),
+            _ptr(bias.padded) if bias is not None else None, bias_len, _stream())
         if kernel in ("mma", "tma"):
             al.sb_attention_force_mma({"mma": 1, "tma": 2}.get(_os.environ.get("SB_ATTN", ""), 0))
         if rc != 0:
@@ -553,7 +570,8 @@ def attention(q: torch.Tensor, out: torch.Tensor, plan, group_index: int, cache:
             _i32(plan.row_pos, "row_pos"), _i32(g.page_off, "page_off"),
             _i32(g.page_ids, "page_ids"), g.page_size, _ptr(cache), _code(cache.dtype),
             n_q_heads, n_kv_heads, head_dim, window, ctypes.c_float(scale), _ptr(sink),
-            ctypes.c_float(softcap), int(chunk), _ptr(bias), bias_len, _stream()), "attention (plain kernel)")
+            ctypes.c_float(softcap), int(chunk), _ptr(bias.values) if bias is not None else None, bias_len, _stream()),
+            "attention (plain kernel)")
     return out
 
 

@@ -189,7 +189,7 @@ class WindowAttention(Mixer):
         if self.taps:
             self.w_conv = _cat([get(p + n + ".conv") for n in (q, k, v)])
         if self.distance_bias:
-            self.bias = bias_by_distance(get(p + self.distance_bias[0]), int(self.distance_bias[1]), self.chunk)
+            self.bias = ops.DistanceBias(bias_by_distance(get(p + self.distance_bias[0]), int(self.distance_bias[1]), self.chunk))
 
     def first_weights(self, rows):
         n, k = self.w_in.shape

@@ -30,14 +30,9 @@ def squared_relu(z):
 
 def short_conv(u, w):
     """y_t = sum_j w[:, j] u_(t - taps + 1 + j) for u [T, channels], zeros before the start."""
-    T, taps = u.shape[0], w.shape[1]
-    y = torch.zeros_like(u)
-    for t in range(T):
-        for j in range(taps):
-            s = t - taps + 1 + j
-            if s >= 0:
-                y[t] += w[:, j] * u[s]
-    return y
+    taps = w.shape[1]
+    padded = torch.cat([torch.zeros(taps - 1, u.shape[1], dtype=F), u])
+    return sum(w[:, j] * padded[j:j + u.shape[0]] for j in range(taps))
 
 
 def bucket(n, rows, most):
@@ -51,12 +46,9 @@ def bucket(n, rows, most):
 
 def distance_bias(T, rel, most):
     """[T, T, heads]: rel[bucket(i - j)] where j <= i, zero elsewhere."""
-    out = torch.zeros(T, T, rel.shape[1], dtype=F)
-    by_distance = torch.stack([rel[bucket(n, rel.shape[0], most)] for n in range(T)])
-    for i in range(T):
-        for j in range(i + 1):
-            out[i, j] = by_distance[i - j]
-    return out
+    rows = torch.tensor([bucket(n, rel.shape[0], most) for n in range(T)])
+    back = torch.arange(T).view(T, 1) - torch.arange(T).view(1, T)
+    return rel[rows[back.clamp(min=0)]] * (back >= 0).unsqueeze(-1)
 
 
 def chunk_mask(T, size):
@@ -120,13 +112,17 @@ def moe_ff(h, get, mlp, gaps=None):
     r = mlp["router"]
     z = h @ get("router").T
     out = torch.zeros_like(h)
+    sent = {}                                   # router output -> [(token, weight)]
     for t in range(h.shape[0]):
         chosen, weights, gap = route(z[t], get("correction"), r)
         if gaps is not None:
             gaps.append(gap)
         for e, w in zip(chosen, weights):
-            y = squared_relu_ff(h[t], lambda n: get(f"e{e}.{n}")) if e < r["experts"] else h[t]
-            out[t] += w * y
+            sent.setdefault(e, []).append((t, w))
+    for e, pairs in sent.items():
+        rows = torch.tensor([t for t, _ in pairs])
+        y = squared_relu_ff(h[rows], lambda n: get(f"e{e}.{n}")) if e < r["experts"] else h[rows]
+        out[rows] += torch.tensor([w for _, w in pairs], dtype=F).view(-1, 1) * y
     if mlp.get("shared") is not None:
         out = out + torch.sigmoid(h @ get("shared.sg").T) * squared_relu_ff(h, lambda n: get("shared." + n))
     return out
