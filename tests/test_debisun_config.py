@@ -91,7 +91,7 @@ def test_errors_name_the_key(edit, key):
     assert key in str(e.value)
 
 
-@pytest.mark.parametrize("rows,most", [(32, 120), (8, 20), (2, 3), (4, 6), (16, 300), (6, 11), (64, 4096)])
+@pytest.mark.parametrize("rows,most", [(32, 150), (8, 20), (2, 3), (4, 6), (16, 300), (6, 11), (64, 4096)])
 def test_distance_buckets(rows, most):
     half = rows // 2
     got = [distance_bucket(n, rows, most) for n in range(2 * most)]
