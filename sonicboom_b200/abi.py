@@ -27,6 +27,8 @@ CORE = {
     "sb_embed": ("i", "pipiiifps"),
     "sb_rmsnorm": ("i", "ppiipifpis"),
     "sb_rmsnorm_ld": ("i", "pipiipifpis"),
+    "sb_rmsnorm_pair": ("i", "piippifppis"),
+    "sb_embed_norm": ("i", "pipiiifpifps"),
     "sb_softcap": ("i", "pzfs"),
     "sb_add_bias": ("i", "ppiiis"),
     "sb_cast": ("i", "pipizs"),
@@ -56,14 +58,15 @@ CORE = {
     "sb_mlstm_scan": ("i", "pippiiippiffipipps"),
     "sb_mlstm_out": ("i", "pppiiiipifpis"),
     "sb_attention_plain": ("i", "ppiippppipiiiiifpfipis"),
-    "sb_stream_add": ("i", "pppiiippifpis"),
+    "sb_stream_add": ("i", "pppiiippifpipps"),
     "sb_polynorm": ("i", "piipifpis"),
     "sb_attn_prep": ("i", "piiiiiiiiiiiippppiiffppppipipiis"),
     "sb_attn_unrotate": ("i", "ppiiiiiipppis"),
+    "sb_attn_gate": ("i", "piiiiipifpiis"),
     "sb_linrec_prep": ("i", "piiiiiiffiipppfppiiis"),
     "sb_linrec_scan": ("i", "piiiipppiippiiipps"),
     "sb_linrec_force_columns": ("v", "i"),
-    "sb_linrec_out": ("i", "ppiiiiipiiifpis"),
+    "sb_linrec_out": ("i", "ppiiiiipiiiffpiiis"),
     "sb_embed_pair": ("i", "pippppppiipiiiifps"),
     "sb_keep_last_token": ("i", "pppips"),
     "sb_layernorm": ("i", "ppiippifpis"),
@@ -72,6 +75,11 @@ CORE = {
     "sb_conv_heads_max_taps": ("i", ""),
     "sb_delta_prep": ("i", "piiiiiiiipppiffps"),
     "sb_delta_scan": ("i", "piiiipippiipps"),
+    "sb_gdelta_step": ("i", "piiiiiiiiiiipppppppffpffpiiis"),
+    "sb_gdelta_mats_floats": ("z", "iii"),
+    "sb_gdelta_prep": ("i", "piiiiiiiiiipppiippppffpps"),
+    "sb_gdelta_scan": ("i", "pppiiiiiiiipppppps"),
+    "sb_gdelta_force_columns": ("v", "i"),
     "sb_ssd_prep": ("i", "piiipiiiiippips"),
     "sb_ssd_out": ("i", "ppiiipiiiiippifpis"),
     "sb_attention_sigmoid": ("i", "ppiippiippppipiiiiiiffps"),
@@ -80,10 +88,11 @@ CORE = {
     "sb_moe_tile_rows": ("i", "iiiii"),
     "sb_moe_max_tiles": ("i", "iii"),
     "sb_moe_group": ("i", "piiipps"),
+    "sb_moe_group_by_token": ("i", "pipiiiippps"),
     "sb_moe_up": ("i", "pipippiiiiiiiffps"),
     "sb_moe_down": ("i", "pipippiiiiiips"),
     "sb_moe_combine": ("i", "pppiiis"),
-    "sb_moe_join": ("i", "ppppipippipiiiipis"),
+    "sb_moe_join": ("i", "ppppfipippipiiiipis"),
     "sb_sample_params_size": ("i", ""),
     "sb_sample": ("i", "piippipps"),
     "sb_add_i32": ("i", "piis"),

@@ -92,6 +92,31 @@ class MefupelLayer:
     mlp: Optional[DenseFFConfig]
 
 
+def loop_config(d: dict, n_layers: int) -> Optional[LoopConfig]:
+    """config.json's `loop` {start, stop, times}, None without one."""
+    loop = d.get("loop")
+    if loop is None:
+        return None
+    if not isinstance(loop, dict):
+        raise ConfigError("missing/invalid config key: loop (expected an object)")
+    loop = LoopConfig(start=_num(loop, "start", "loop.", positive=False),
+                      stop=_num(loop, "stop", "loop.", positive=False), times=_num(loop, "times", "loop."))
+    if not 0 <= loop.start <= loop.stop <= n_layers:
+        raise ConfigError(f"missing/invalid config key: loop ({loop.start} .. {loop.stop} is no "
+                          f"stretch of the {n_layers} layers)")
+    return loop
+
+
+def loop_order(n_layers: int, loop: Optional[LoopConfig]) -> list:
+    """(layer, pass number or None) in run order; a number marks the first layer of a pass."""
+    if loop is None or loop.start == loop.stop:
+        return [(i, None) for i in range(n_layers)]
+    order = [(i, None) for i in range(loop.start)]
+    for t in range(loop.times):
+        order += [(i, t if i == loop.start else None) for i in range(loop.start, loop.stop)]
+    return order + [(i, None) for i in range(loop.stop, n_layers)]
+
+
 def _rot(m: dict, where: str, dim: int):
     rot = _sub(m, "rot", where)
     base, dims = _num(rot, "base", where + "rot.", float), _num(rot, "dims", where + "rot.", positive=False)
@@ -175,16 +200,7 @@ class MefupelConfig:
                                       f"{mlp.get('kind') if isinstance(mlp, dict) else mlp!r} (only 'dense')")
                 mlp = DenseFFConfig(ff=_num(mlp, "ff", w + "mlp."))
             layers.append(MefupelLayer(kind, mixer, mlp))
-        loop = d.get("loop")
-        if loop is not None:
-            if not isinstance(loop, dict):
-                raise ConfigError("missing/invalid config key: loop (expected an object)")
-            loop = LoopConfig(start=_num(loop, "start", "loop.", positive=False),
-                              stop=_num(loop, "stop", "loop.", positive=False), times=_num(loop, "times", "loop."))
-            if not 0 <= loop.start <= loop.stop <= len(layers):
-                raise ConfigError(f"missing/invalid config key: loop ({loop.start} .. {loop.stop} is no "
-                                  f"stretch of the {len(layers)} layers)")
-        return cls(vocab=vocab, width=width, eps=eps, layers=tuple(layers), loop=loop)
+        return cls(vocab=vocab, width=width, eps=eps, layers=tuple(layers), loop=loop_config(d, len(layers)))
 
     def to_dict(self) -> dict:
         """config.json content that `from_dict` reads back to an equal configuration."""
@@ -214,14 +230,7 @@ class MefupelConfig:
         return d
 
     def run_order(self) -> list:
-        """(layer, pass number or None) in run order; a number marks the first layer of a pass."""
-        n, loop = len(self.layers), self.loop
-        if loop is None or loop.start == loop.stop:
-            return [(i, None) for i in range(n)]
-        order = [(i, None) for i in range(loop.start)]
-        for t in range(loop.times):
-            order += [(i, t if i == loop.start else None) for i in range(loop.start, loop.stop)]
-        return order + [(i, None) for i in range(loop.stop, n)]
+        return loop_order(len(self.layers), self.loop)
 
     def to_spec(self) -> ModelSpec:
         """The model as parts: one block per layer in which mixer and feed-forward read the same

@@ -178,6 +178,7 @@ class ModelSpec:
     unused_tensors: tuple = ()          # (name, shape) of tensors a file may hold that nothing reads
     pair_embedding: Optional[PairEmbeddingSpec] = None   # added to every embedding row
     side_table: Optional[SideTableSpec] = None           # read by the layers that have a side input
+    embedding_norm: Optional[NormSpec] = None            # norms every embedding row before the first layer
 
     def validate(self) -> None:
         if not self.layers:

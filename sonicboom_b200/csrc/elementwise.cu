@@ -49,11 +49,12 @@ extern "C" int sb_embed(const int32_t* tokens, int n_rows, const void* table, in
 // (core/src/nn/norm.cpp:25-42, core/src/nn/cuda_elementwise.cu:684-711).  One block per row;
 // the sum is a fixed tree (thread-strided partial sums, warp shuffles, then the warps in
 // order), so a row's result does not depend on which other rows are in the launch.
-// `rows`, when given, gathers: output row r is the norm of input row rows[r].
+// `rows`, when given, gathers: output row r is the norm of input row rows[r].  `w2` / `out2`, when given: the
+// same row with a second weight.
 template <typename TW, typename TO>
 __global__ void rmsnorm_kernel(const float* x, size_t x_ld, const int32_t* rows,
                                const TW* __restrict__ w, int width, float eps,
-                               TO* __restrict__ out) {
+                               TO* __restrict__ out, const TW* __restrict__ w2, TO* __restrict__ out2) {
   __shared__ float warp_sums[32];
   __shared__ float inv_shared;
   sb_pdl_launch();
@@ -77,8 +78,10 @@ __global__ void rmsnorm_kernel(const float* x, size_t x_ld, const int32_t* rows,
   __syncthreads();
   const float inv = inv_shared;
   TO* o = out + (size_t)r * width;
-  for (int i = threadIdx.x; i < width; i += blockDim.x)
+  for (int i = threadIdx.x; i < width; i += blockDim.x) {
     o[i] = sb_from_f32<TO>((xr[i] * inv) * sb_to_f32<TW>(w[i]));
+    if (w2) out2[(size_t)r * width + i] = sb_from_f32<TO>((xr[i] * inv) * sb_to_f32<TW>(w2[i]));
+  }
 }
 
 // The same for widths that are multiples of 4 and at most 4096: every thread keeps its part of the
@@ -117,7 +120,7 @@ constexpr int NORM_THREADS = 256, NORM_VEC = 4;      // 256 threads x 4 vectors 
 template <typename TW, typename TO>
 __global__ void __launch_bounds__(NORM_THREADS)
 rmsnorm_vec_kernel(const float* x, size_t x_ld, const int32_t* rows, const TW* __restrict__ w, int width,
-                   float eps, TO* __restrict__ out) {
+                   float eps, TO* __restrict__ out, const TW* __restrict__ w2, TO* __restrict__ out2) {
   __shared__ float warp_sums[NORM_THREADS / 32];
   __shared__ float inv_shared;
   sb_pdl_launch();
@@ -156,6 +159,12 @@ rmsnorm_vec_kernel(const float* x, size_t x_ld, const int32_t* rows, const TW* _
 #pragma unroll
       for (int j = 0; j < 4; ++j) y[j] = (v[i][j] * inv) * wv[j];
       sb_store4<TO>(o + e, y);
+      if (w2) {
+        sb_load4<TW>(w2 + e, wv);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) y[j] = (v[i][j] * inv) * wv[j];
+        sb_store4<TO>(out2 + (size_t)r * width + e, y);
+      }
     }
   }
 }
@@ -166,10 +175,10 @@ extern "C" int sb_rmsnorm(const float* x, const int32_t* rows, int n_rows, int w
   return sb_rmsnorm_ld(x, width, rows, n_rows, width, weight, weight_dtype, eps, out, out_dtype, stream);
 }
 
-// The same over the first `width` values of input rows that lie `x_ld` values apart.
-extern "C" int sb_rmsnorm_ld(const float* x, int x_ld, const int32_t* rows, int n_rows, int width,
-                             const void* weight, int weight_dtype, float eps, void* out,
-                             int out_dtype, cudaStream_t stream) {
+// Input rows lie `x_ld` values apart; their first `width` values are normed.
+static int rmsnorm_run(const float* x, int x_ld, const int32_t* rows, int n_rows, int width, const void* weight,
+                       int weight_dtype, float eps, void* out, int out_dtype, const void* weight2, void* out2,
+                       cudaStream_t stream) {
   if (n_rows <= 0 || width <= 0 || x_ld < width)
     SB_FAIL(SB_ERR_ARG, "sb_rmsnorm: n_rows=%d width=%d rows %d apart", n_rows, width, x_ld);
   if (!sb_valid_dtype(weight_dtype) || !sb_valid_dtype(out_dtype))
@@ -177,19 +186,80 @@ extern "C" int sb_rmsnorm_ld(const float* x, int x_ld, const int32_t* rows, int 
   if (!(eps >= 0.0f)) SB_FAIL(SB_ERR_ARG, "sb_rmsnorm: eps %g", eps);
   const int threads = width >= 2048 ? 512 : (width >= 512 ? 256 : 128);
   const bool vec = width % 4 == 0 && x_ld % 4 == 0 && width <= NORM_THREADS * NORM_VEC * 4 &&
-                   (((uintptr_t)x | (uintptr_t)weight | (uintptr_t)out) & 15) == 0;
+                   (((uintptr_t)x | (uintptr_t)weight | (uintptr_t)out | (uintptr_t)weight2 | (uintptr_t)out2) & 15) == 0;
   SB_DISPATCH_DTYPE(weight_dtype, TW, {
     SB_DISPATCH_DTYPE(out_dtype, TO, {
       if (vec)
         sb_launch<SB_K_ELEMENTWISE>(rmsnorm_vec_kernel<TW, TO>, dim3(n_rows), dim3(NORM_THREADS), 0, stream, x,
                   (size_t)x_ld, rows,
-                  (const TW*)weight, width, eps, (TO*)out);
+                  (const TW*)weight, width, eps, (TO*)out, (const TW*)weight2, (TO*)out2);
       else
         sb_launch<SB_K_ELEMENTWISE>(rmsnorm_kernel<TW, TO>, dim3(n_rows), dim3(threads), 0, stream, x, (size_t)x_ld, rows,
-                  (const TW*)weight, width, eps, (TO*)out);
+                  (const TW*)weight, width, eps, (TO*)out, (const TW*)weight2, (TO*)out2);
     });
   });
   SB_CHECK_LAUNCH("sb_rmsnorm");
+  return SB_OK;
+}
+
+extern "C" int sb_rmsnorm_ld(const float* x, int x_ld, const int32_t* rows, int n_rows, int width,
+                             const void* weight, int weight_dtype, float eps, void* out,
+                             int out_dtype, cudaStream_t stream) {
+  return rmsnorm_run(x, x_ld, rows, n_rows, width, weight, weight_dtype, eps, out, out_dtype, nullptr, nullptr, stream);
+}
+
+// One reading of the row for two norms that share eps and differ in the weight (both of one dtype).
+extern "C" int sb_rmsnorm_pair(const float* x, int n_rows, int width, const void* weight1, const void* weight2,
+                               int weight_dtype, float eps, void* out1, void* out2, int out_dtype, cudaStream_t stream) {
+  if (!weight2 || !out2) SB_FAIL(SB_ERR_ARG, "sb_rmsnorm_pair: the second norm's weight or result is missing");
+  return rmsnorm_run(x, width, nullptr, n_rows, width, weight1, weight_dtype, eps, out1, out_dtype, weight2, out2, stream);
+}
+
+// The embedding row, times `scale`, RMS-normed with the weight `w`: what a model hands its first layer when it norms its
+// embeddings.  An id outside the table gives a row of NaN.
+template <typename TW, typename TN>
+__global__ void __launch_bounds__(256)
+embed_norm_kernel(const int32_t* tokens, const TW* __restrict__ table, int vocab, int width, float scale,
+                  const TN* __restrict__ w, float eps, float* __restrict__ out) {
+  __shared__ float warp_sums[8];
+  sb_pdl_launch();
+  sb_pdl_wait();
+  const int t = blockIdx.x, id = tokens[t];
+  float* o = out + (size_t)t * width;
+  if ((unsigned)id >= (unsigned)vocab) {
+    for (int i = threadIdx.x; i < width; i += 256) o[i] = __int_as_float(0x7fc00000);
+    return;
+  }
+  const TW* row = table + (size_t)id * width;
+  float s = 0.0f;
+  for (int i = threadIdx.x; i < width; i += 256) {
+    const float v = sb_to_f32<TW>(row[i]) * scale;
+    o[i] = v;
+    s = fmaf(v, v, s);
+  }
+  s = sb_warp_sum(s);
+  if ((threadIdx.x & 31) == 0) warp_sums[threadIdx.x >> 5] = s;
+  __syncthreads();
+  float total = 0.0f;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) total += warp_sums[i];
+  const float inv = 1.0f / sqrtf(total / (float)width + eps);
+  for (int i = threadIdx.x; i < width; i += 256) o[i] = (o[i] * inv) * sb_to_f32<TN>(w[i]);   // a thread reads what it wrote itself
+}
+
+extern "C" int sb_embed_norm(const int32_t* tokens, int n_rows, const void* table, int table_dtype, int vocab, int width,
+                             float scale, const void* weight, int weight_dtype, float eps, float* out, cudaStream_t stream) {
+  if (n_rows <= 0 || width <= 0 || vocab <= 0 || !tokens || !table || !weight || !out)
+    SB_FAIL(SB_ERR_ARG, "sb_embed_norm: n_rows=%d vocab=%d width=%d", n_rows, vocab, width);
+  if (!sb_valid_dtype(table_dtype) || !sb_valid_dtype(weight_dtype) || !(eps >= 0.0f))
+    SB_FAIL(SB_ERR_ARG, "sb_embed_norm: dtype codes %d %d, eps %g", table_dtype, weight_dtype, eps);
+  SB_DISPATCH_DTYPE(table_dtype, TW, {
+    SB_DISPATCH_DTYPE(weight_dtype, TN, {
+      sb_launch<SB_K_ELEMENTWISE>(embed_norm_kernel<TW, TN>, dim3(n_rows), dim3(256), 0, stream, tokens, (const TW*)table, vocab,
+                                  width, scale, (const TN*)weight, eps, out);
+    });
+  });
+  SB_CHECK_LAUNCH("sb_embed_norm");
   return SB_OK;
 }
 

@@ -755,7 +755,7 @@ __device__ __forceinline__ void rn_store4(bf16* p, const float (&v)[4]) {
 template <typename TW, typename TN>
 __global__ void __launch_bounds__(RN_THREADS)
 tc5_reduce_norm_kernel(const Tc5Params p, int bn, const TW* __restrict__ norm_w, float eps,
-                       TN* __restrict__ norm_out) {
+                       TN* __restrict__ norm_out, const TW* __restrict__ norm_w2, TN* __restrict__ norm_out2) {
   namespace cg = cooperative_groups;
   cg::cluster_group cluster = cg::this_cluster();
   __shared__ float warp_sums[RN_THREADS / 32];
@@ -825,6 +825,12 @@ tc5_reduce_norm_kernel(const Tc5Params p, int bn, const TW* __restrict__ norm_w,
 #pragma unroll
     for (int k = 0; k < 4; ++k) y[k] = (v[i][k] * inv) * wv[i][k];
     rn_store4(norm_out + (size_t)j * p.N + (size_t)g * 4, y);
+    if (norm_w2) {                                   // the same rows with a second weight
+      rn_load4(norm_w2 + (size_t)g * 4, wv[i]);
+#pragma unroll
+      for (int k = 0; k < 4; ++k) y[k] = (v[i][k] * inv) * wv[i][k];
+      rn_store4(norm_out2 + (size_t)j * p.N + (size_t)g * 4, y);
+    }
   }
 }
 
@@ -1119,17 +1125,21 @@ static int tc5_run(const void* A, int a_dtype, const void* W, int w_dtype, int M
   if (norm) {
     if (epilogue == SB_EPI_SWIGLU || epilogue == SB_EPI_RELU2 || out_dtype != SB_F32)
       SB_FAIL(SB_ERR_UNSUPPORTED, "sb_gemm_tc5: a norm follows a float32 product without an activation");
-    if (!norm->norm_out || !sb_valid_dtype(norm->norm_weight_dtype) ||
+    if (!norm->norm_out || (norm->norm_weight2 == nullptr) != (norm->norm_out2 == nullptr) || !sb_valid_dtype(norm->norm_weight_dtype) ||
         !sb_valid_dtype(norm->norm_out_dtype) || !(norm->norm_eps >= 0.0f))
       SB_FAIL(SB_ERR_ARG, "sb_gemm_tc5: norm output, dtype codes %d %d or eps %g",
               norm->norm_weight_dtype, norm->norm_out_dtype, norm->norm_eps);
     if (!norm_fuses(M, N, K, n_sms, epilogue, out_dtype, form) ||
-        (((uintptr_t)norm->norm_weight | (uintptr_t)norm->norm_out | (uintptr_t)out |
+        (((uintptr_t)norm->norm_weight | (uintptr_t)norm->norm_out | (uintptr_t)norm->norm_weight2 |
+          (uintptr_t)norm->norm_out2 | (uintptr_t)out |
           (uintptr_t)residual | (uintptr_t)bias) & 15)) {
       // the product as usual, then the norm as a kernel of its own
       if (int rc = tc5_run(A, a_dtype, W, w_dtype, M, N, K, epilogue, bias, bias_dtype, residual,
                            out, out_dtype, scratch, scratch_bytes, n_sms, form, nullptr, stream))
         return rc;
+      if (norm->norm_weight2)
+        return sb_rmsnorm_pair((const float*)out, M, N, norm->norm_weight, norm->norm_weight2, norm->norm_weight_dtype,
+                               norm->norm_eps, norm->norm_out, norm->norm_out2, norm->norm_out_dtype, stream);
       return sb_rmsnorm((const float*)out, nullptr, M, N, norm->norm_weight, norm->norm_weight_dtype,
                         norm->norm_eps, norm->norm_out, norm->norm_out_dtype, stream);
     }
@@ -1294,7 +1304,7 @@ static int tc5_run(const void* A, int a_dtype, const void* W, int w_dtype, int M
     SB_DISPATCH_DTYPE(norm->norm_weight_dtype, TW, {
       SB_DISPATCH_DTYPE(norm->norm_out_dtype, TN, {
         cudaLaunchKernelEx(&cfg, tc5_reduce_norm_kernel<TW, TN>, p, bn, (const TW*)norm->norm_weight,
-                           norm->norm_eps, (TN*)norm->norm_out);
+                           norm->norm_eps, (TN*)norm->norm_out, (const TW*)norm->norm_weight2, (TN*)norm->norm_out2);
       });
     });
     SB_CHECK_LAUNCH("sb_gemm_tc5 (reduce + norm)");

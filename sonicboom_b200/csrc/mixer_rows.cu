@@ -8,6 +8,8 @@
 //                      (2i, 2i + 1), values that are the raw key projection, values rotated by their
 //                      own position, heads padded with zeros to the cache's head size
 //   sb_attn_unrotate:  attention results turned back by the query's position, padding dropped
+//   sb_attn_gate:      attention results with the padding dropped, every value times the logistic function of
+//                      its own gate value and a constant, into columns of a wider row
 //   sb_linrec_prep:    rotation and scaling of a recurrence's q and k in place; decay logits to
 //                      decays exp(logsigmoid(z) / tau) in place
 //   sb_linrec_out:     RMS norm of every head's recurrence output, optional weight, gate silu(g)
@@ -40,7 +42,7 @@ __device__ __forceinline__ float block_sum(float s, float* red) {
 template <int NT, typename TV, typename TN, typename TO>
 __global__ void __launch_bounds__(NT)
 stream_add_kernel(const float* x, const float* add, const TV* __restrict__ vec, int width, float* out,
-                  const TN* __restrict__ next_w, float next_eps, TO* normed) {
+                  const TN* __restrict__ next_w, float next_eps, TO* normed, const TN* __restrict__ next_w2, TO* normed2) {
   __shared__ float red[NT / 32 + 1];
   sb_pdl_launch();
   sb_pdl_wait();
@@ -55,8 +57,10 @@ stream_add_kernel(const float* x, const float* add, const TV* __restrict__ vec, 
   }
   if (!normed) return;
   const float inv = 1.0f / sqrtf(block_sum<NT>(sq, red) / (float)width + next_eps);
-  for (int i = threadIdx.x; i < width; i += NT)
+  for (int i = threadIdx.x; i < width; i += NT) {
     normed[r * width + i] = sb_from_f32<TO>((out[r * width + i] * inv) * sb_to_f32<TN>(next_w[i]));
+    if (next_w2) normed2[r * width + i] = sb_from_f32<TO>((out[r * width + i] * inv) * sb_to_f32<TN>(next_w2[i]));
+  }
 }
 
 // -------------------------------------------------------------------------------- polynorm
@@ -325,6 +329,53 @@ attn_unrotate_kernel(const T* in, T* out, int n_heads, int hd, int vdim, int int
                  });
 }
 
+// A thread takes V neighbouring values of a head's result.
+template <int V, typename T>
+__global__ void __launch_bounds__(256)
+attn_gate_kernel(const T* in, T* out, size_t n, int per_row, int hd, int vdim, const float* gate, int gate_ld, float scale,
+                 int ld_out) {
+  sb_pdl_launch();
+  sb_pdl_wait();
+  for (size_t e = (size_t)blockIdx.x * 256 + threadIdx.x; e < n; e += (size_t)gridDim.x * 256) {
+    const size_t t = e / per_row;
+    const int at = (int)(e % per_row) * V, h = at / vdim, c = at - h * vdim;
+    const T* src = in + (t * (per_row * V / vdim) + h) * hd + c;
+    const float* g = gate ? gate + t * gate_ld + at : nullptr;
+    T* dst = out + t * ld_out + at;
+    if constexpr (V == 4) {
+      float v[4], z[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+      if constexpr (sizeof(T) == 2) {
+        const uint2 u = *reinterpret_cast<const uint2*>(src);
+        const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+        const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+        v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
+      } else {
+        const float4 f = *reinterpret_cast<const float4*>(src);
+        v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+      }
+      if (g) {
+        const float4 f = *reinterpret_cast<const float4*>(g);
+        z[0] = f.x; z[1] = f.y; z[2] = f.z; z[3] = f.w;
+      }
+#pragma unroll
+      for (int j = 0; j < 4; ++j) v[j] = (g ? v[j] / (1.0f + expf(-z[j])) : v[j]) * scale;
+      if constexpr (sizeof(T) == 2) {
+        __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
+        uint2 u;
+        u.x = *reinterpret_cast<uint32_t*>(&a);
+        u.y = *reinterpret_cast<uint32_t*>(&b);
+        *reinterpret_cast<uint2*>(dst) = u;
+      } else {
+        *reinterpret_cast<float4*>(dst) = make_float4(v[0], v[1], v[2], v[3]);
+      }
+    } else {
+      float v = sb_to_f32<T>(src[0]);
+      if (g) v = v / (1.0f + expf(-g[0]));
+      dst[0] = sb_from_f32<T>(v * scale);
+    }
+  }
+}
+
 // ---------------------------------------------------------------------- linear recurrence
 // With `a2` the decay logits are worked out here: z[t, c] = bias[c] + sum_r a2[c, r] * proj[t, a1_off + r]
 // (r ascending, float32), the second half of a low-rank map whose first half came with the projection.
@@ -376,11 +427,11 @@ __global__ void linrec_prep_kernel(float* proj, int ld, int q_off, int k_off, in
   }
 }
 
-// One warp per (row, head).
+// One warp per (row, head); a row's results start at column out_off of a row of ld_out.
 template <typename TW, typename TO>
 __global__ void linrec_out_kernel(const float* o, const float* proj, int ld, int g_off, size_t n_items,
                                   int n_heads, int vdim, const TW* __restrict__ norm_w, int w_per_head,
-                                  int gate_sigmoid, float eps, TO* out) {
+                                  int gate_sigmoid, float eps, float scale, TO* out, int ld_out, int out_off) {
   sb_pdl_launch();
   sb_pdl_wait();
   const int lane = threadIdx.x & 31;
@@ -396,7 +447,8 @@ __global__ void linrec_out_kernel(const float* o, const float* proj, int ld, int
   for (int j = lane; j < vdim; j += 32) {
     float v = src[j] * inv;
     if (norm_w) v *= sb_to_f32<TW>(norm_w[(w_per_head ? (size_t)h * vdim : 0) + j]);
-    out[item * vdim + j] = sb_from_f32<TO>(gate_sigmoid ? v / (1.0f + expf(-g[j])) : v * sb_silu(g[j]));
+    v = gate_sigmoid ? v / (1.0f + expf(-g[j])) : v * sb_silu(g[j]);
+    out[t * ld_out + out_off + (size_t)h * vdim + j] = sb_from_f32<TO>(scale == 1.0f ? v : v * scale);
   }
 }
 
@@ -409,7 +461,9 @@ inline int grid_for(size_t n, int threads) {
 
 extern "C" int sb_stream_add(const float* x, const float* add, const void* vec, int vec_dtype, int n_rows,
                              int width, float* out, const void* next_w, int next_w_dtype, float next_eps,
-                             void* normed, int normed_dtype, cudaStream_t stream) {
+                             void* normed, int normed_dtype, const void* next_w2, void* normed2, cudaStream_t stream) {
+  if ((next_w2 == nullptr) != (normed2 == nullptr) || (next_w2 && !normed))
+    SB_FAIL(SB_ERR_ARG, "sb_stream_add: a second norm comes with a first one, a weight and a result");
   if (n_rows <= 0 || width <= 0 || !x || !out) SB_FAIL(SB_ERR_ARG, "sb_stream_add: rows=%d width=%d", n_rows, width);
   if ((vec && !sb_valid_dtype(vec_dtype)) || (normed && (!next_w || !sb_valid_dtype(next_w_dtype) || !sb_valid_dtype(normed_dtype))))
     SB_FAIL(SB_ERR_ARG, "sb_stream_add: dtype codes %d %d %d", vec_dtype, next_w_dtype, normed_dtype);
@@ -419,10 +473,12 @@ extern "C" int sb_stream_add(const float* x, const float* add, const void* vec, 
       SB_DISPATCH_DTYPE(normed ? normed_dtype : SB_F32, TO, {
         if (n_rows >= 512 || width <= 1024)
           sb_launch<SB_K_ELEMENTWISE>(stream_add_kernel<256, TV, TN, TO>, dim3(n_rows), dim3(256), 0, stream, x, add,
-                                      (const TV*)vec, width, out, (const TN*)next_w, next_eps, (TO*)normed);
+                                      (const TV*)vec, width, out, (const TN*)next_w, next_eps, (TO*)normed,
+                                      (const TN*)next_w2, (TO*)normed2);
         else
           sb_launch<SB_K_ELEMENTWISE>(stream_add_kernel<1024, TV, TN, TO>, dim3(n_rows), dim3(1024), 0, stream, x, add,
-                                      (const TV*)vec, width, out, (const TN*)next_w, next_eps, (TO*)normed);
+                                      (const TV*)vec, width, out, (const TN*)next_w, next_eps, (TO*)normed,
+                                      (const TN*)next_w2, (TO*)normed2);
       });
     });
   });
@@ -514,6 +570,29 @@ extern "C" int sb_attn_unrotate(const void* in, void* out, int dtype, int n_rows
   return SB_OK;
 }
 
+extern "C" int sb_attn_gate(const void* in, int dtype, int n_rows, int n_heads, int hd, int vdim, const float* gate, int gate_ld,
+                            float scale, void* out, int ld_out, int out_off, cudaStream_t stream) {
+  if (n_rows <= 0 || n_heads <= 0 || vdim <= 0 || hd < vdim || !in || !out || !sb_valid_dtype(dtype))
+    SB_FAIL(SB_ERR_ARG, "sb_attn_gate: rows=%d heads=%d hd=%d vdim=%d dtype=%d", n_rows, n_heads, hd, vdim, dtype);
+  if (out_off < 0 || out_off + n_heads * vdim > ld_out)
+    SB_FAIL(SB_ERR_ARG, "sb_attn_gate: %d values at column %d of %d", n_heads * vdim, out_off, ld_out);
+  const bool vec = vdim % 4 == 0 && hd % 4 == 0 && ld_out % 4 == 0 && out_off % 4 == 0 && gate_ld % 4 == 0 &&
+                   (((uintptr_t)in | (uintptr_t)out | (uintptr_t)gate) & 15) == 0;
+  const int per_row = n_heads * vdim / (vec ? 4 : 1);
+  const size_t n = (size_t)n_rows * per_row;
+  SB_DISPATCH_DTYPE(dtype, T, {
+    T* o = (T*)out + out_off;
+    if (vec)
+      sb_launch<SB_K_ELEMENTWISE>(attn_gate_kernel<4, T>, dim3(grid_for(n, 256)), dim3(256), 0, stream, (const T*)in, o, n,
+                                  per_row, hd, vdim, gate, gate_ld, scale, ld_out);
+    else
+      sb_launch<SB_K_ELEMENTWISE>(attn_gate_kernel<1, T>, dim3(grid_for(n, 256)), dim3(256), 0, stream, (const T*)in, o, n,
+                                  per_row, hd, vdim, gate, gate_ld, scale, ld_out);
+  });
+  SB_CHECK_LAUNCH("sb_attn_gate");
+  return SB_OK;
+}
+
 extern "C" int sb_linrec_prep(float* proj, int n_rows, int ld, int q_off, int k_off, int n_heads, int dim,
                               float q_scale, float k_scale, int rot, int interleaved, const float* inv_freq,
                               const int32_t* row_pos, float* z, float inv_tau, const void* a2,
@@ -535,7 +614,9 @@ extern "C" int sb_linrec_prep(float* proj, int n_rows, int ld, int q_off, int k_
 
 extern "C" int sb_linrec_out(const float* o, const float* proj, int n_rows, int ld, int g_off, int n_heads,
                              int vdim, const void* norm_w, int norm_w_dtype, int w_per_head, int gate_sigmoid,
-                             float eps, void* out, int out_dtype, cudaStream_t stream) {
+                             float eps, float scale, void* out, int out_dtype, int ld_out, int out_off, cudaStream_t stream) {
+  if (out_off < 0 || (long long)out_off + (long long)n_heads * vdim > ld_out)
+    SB_FAIL(SB_ERR_ARG, "sb_linrec_out: %d heads of %d at column %d of %d", n_heads, vdim, out_off, ld_out);
   if (n_rows <= 0 || n_heads <= 0 || vdim <= 0 || !o || !proj || !out)
     SB_FAIL(SB_ERR_ARG, "sb_linrec_out: rows=%d heads=%d vdim=%d", n_rows, n_heads, vdim);
   if (!sb_valid_dtype(out_dtype) || (norm_w && !sb_valid_dtype(norm_w_dtype)))
@@ -545,7 +626,7 @@ extern "C" int sb_linrec_out(const float* o, const float* proj, int n_rows, int 
   SB_DISPATCH_DTYPE(norm_w ? norm_w_dtype : SB_F32, TW, {
     SB_DISPATCH_DTYPE(out_dtype, TO, {
       sb_launch<SB_K_ELEMENTWISE>(linrec_out_kernel<TW, TO>, dim3(blocks), dim3(256), 0, stream, o, proj, ld, g_off,
-                                  items, n_heads, vdim, (const TW*)norm_w, w_per_head, gate_sigmoid, eps, (TO*)out);
+                                  items, n_heads, vdim, (const TW*)norm_w, w_per_head, gate_sigmoid, eps, scale, (TO*)out, ld_out, out_off);
     });
   });
   SB_CHECK_LAUNCH("sb_linrec_out");

@@ -4,6 +4,7 @@
 //                   over the chosen ones only; expert ids and weights per (row, choice) pair
 //   sb_moe_group:   the pairs grouped by expert, and the tiles of up to `tile_rows` pairs of one expert
 //                   that the products walk (one block; everything stays on the device)
+//   sb_moe_group_by_token: the same where a table names every token id's experts and no router runs
 //   sb_moe_up:      for every tile, gate and up products of the expert with the clamped gated
 //                   activation a * sigmoid(slope a) * (b + 1) in the epilogue.  bfloat16 with inner
 //                   sizes in multiples of 8 runs on tensor cores (mma.sync m16n8k16, tiles of 64 or
@@ -228,8 +229,11 @@ moe_route_scored_kernel(const float* logits, int ld, const float* __restrict__ c
 
 // Pairs whose id is n_experts or more (identity outputs) have no expert and are left out.
 // meta: [0] number of tiles; then per tile (expert, first place in `order`, pairs).
+// With `table` [vocab, top] there is no router: pair p is choice p % top of row p / top, whose token's row of the
+// table names its experts; the ids are written first (a token outside the table: no expert).
 __global__ void __launch_bounds__(1024)
-moe_group_kernel(const int32_t* ids, int n_pairs, int n_experts, int tile_rows, int32_t* order, int32_t* meta) {
+moe_group_kernel(int32_t* ids, int n_pairs, int n_experts, int tile_rows, int32_t* order, int32_t* meta,
+                 const int32_t* tokens, const int32_t* __restrict__ table, int vocab, int top) {
   extern __shared__ int32_t sh[];               // counts, then starts, then cursors
   int32_t* count = sh;
   int32_t* start = sh + n_experts;
@@ -238,7 +242,13 @@ moe_group_kernel(const int32_t* ids, int n_pairs, int n_experts, int tile_rows, 
   for (int e = threadIdx.x; e < n_experts; e += blockDim.x) count[e] = cursor[e] = 0;
   __syncthreads();
   sb_pdl_wait();
-  for (int p = threadIdx.x; p < n_pairs; p += blockDim.x)
+  if (table)
+    for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) {
+      const int tok = tokens[p / top];
+      const int e = (unsigned)tok < (unsigned)vocab ? table[(size_t)tok * top + p % top] : n_experts;
+      ids[p] = (unsigned)e < (unsigned)n_experts ? e : n_experts;
+    }
+  for (int p = threadIdx.x; p < n_pairs; p += blockDim.x)      // a thread reads the ids that it wrote itself
     if (ids[p] < n_experts) atomicAdd(&count[ids[p]], 1);
   __syncthreads();
   if (threadIdx.x == 0) {
@@ -568,7 +578,7 @@ __device__ __forceinline__ Lanes<V> load_lanes(const T* p) {
 
 template <int V, typename TH, typename TS, typename TC>
 __global__ void __launch_bounds__(256)
-moe_join_kernel(float* x, const float* pair_out, const int32_t* ids, const float* weights, int n_experts,
+moe_join_kernel(float* x, const float* pair_out, const int32_t* ids, const float* weights, float weight, int n_experts,
                 const TH* h, const float* shared, const float* gate, int gate_ld, const TS* __restrict__ scale,
                 int top, int width, TC* copy) {
   sb_pdl_launch();
@@ -582,7 +592,7 @@ moe_join_kernel(float* x, const float* pair_out, const int32_t* ids, const float
     const Lanes<V> own = load_lanes<V>(h + r * width + c);
 #pragma unroll 4
     for (int k = 0; k < top; ++k) {
-      const float wk = weights[r * top + k];
+      const float wk = weights ? weights[r * top + k] : weight;
       const Lanes<V> y = ids[r * top + k] < n_experts ? load_lanes<V>(pair_out + (r * top + k) * width + c) : own;
 #pragma unroll
       for (int i = 0; i < V; ++i) s.v[i] = fmaf(wk, y.v[i], s.v[i]);
@@ -675,9 +685,23 @@ extern "C" int sb_moe_group(const int32_t* ids, int n_pairs, int n_experts, int 
     SB_FAIL(SB_ERR_ARG, "sb_moe_group: pairs=%d experts=%d tile_rows=%d", n_pairs, n_experts, tile_rows);
   const size_t smem = (size_t)3 * n_experts * sizeof(int32_t);
   if (smem > 48 * 1024) SB_FAIL(SB_ERR_UNSUPPORTED, "sb_moe_group: %d experts", n_experts);
-  sb_launch<SB_K_ELEMENTWISE>(moe_group_kernel, dim3(1), dim3(1024), smem, stream, ids, n_pairs, n_experts, tile_rows,
-                              order, meta);
+  sb_launch<SB_K_ELEMENTWISE>(moe_group_kernel, dim3(1), dim3(1024), smem, stream, const_cast<int32_t*>(ids), n_pairs,
+                              n_experts, tile_rows, order, meta, (const int32_t*)nullptr, (const int32_t*)nullptr, 0, 1);
   SB_CHECK_LAUNCH("sb_moe_group");
+  return SB_OK;
+}
+
+extern "C" int sb_moe_group_by_token(const int32_t* tokens, int n_rows, const int32_t* table, int vocab, int top, int n_experts,
+                                     int tile_rows, int32_t* ids, int32_t* order, int32_t* meta, cudaStream_t stream) {
+  if (n_rows <= 0 || top <= 0 || vocab <= 0 || n_experts <= 0 || !tokens || !table || !ids || !order || !meta ||
+      (tile_rows != BM && tile_rows != 64 && tile_rows != 128))
+    SB_FAIL(SB_ERR_ARG, "sb_moe_group_by_token: rows=%d top=%d vocab=%d experts=%d tile_rows=%d", n_rows, top, vocab, n_experts,
+            tile_rows);
+  const size_t smem = (size_t)3 * n_experts * sizeof(int32_t);
+  if (smem > 48 * 1024) SB_FAIL(SB_ERR_UNSUPPORTED, "sb_moe_group_by_token: %d experts", n_experts);
+  sb_launch<SB_K_ELEMENTWISE>(moe_group_kernel, dim3(1), dim3(1024), smem, stream, ids, n_rows * top, n_experts, tile_rows, order,
+                              meta, tokens, table, vocab, top);
+  SB_CHECK_LAUNCH("sb_moe_group_by_token");
   return SB_OK;
 }
 
@@ -753,11 +777,11 @@ extern "C" int sb_moe_combine(float* x, const float* pair_out, const float* weig
   return SB_OK;
 }
 
-extern "C" int sb_moe_join(float* x, const float* pair_out, const int32_t* ids, const float* weights, int n_experts,
+extern "C" int sb_moe_join(float* x, const float* pair_out, const int32_t* ids, const float* weights, float weight, int n_experts,
                            const void* h, int h_dtype, const float* shared, const float* gate, int gate_ld,
                            const void* scale, int scale_dtype, int n_rows, int top, int width, void* copy,
                            int copy_dtype, cudaStream_t stream) {
-  if (n_rows <= 0 || top <= 0 || width <= 0 || n_experts <= 0 || !x || !pair_out || !ids || !weights || !h)
+  if (n_rows <= 0 || top <= 0 || width <= 0 || n_experts <= 0 || !x || !pair_out || !ids || !h)
     SB_FAIL(SB_ERR_ARG, "sb_moe_join: rows=%d top=%d width=%d experts=%d", n_rows, top, width, n_experts);
   if (!sb_valid_dtype(h_dtype) || (scale && !sb_valid_dtype(scale_dtype)) || (copy && !sb_valid_dtype(copy_dtype)))
     SB_FAIL(SB_ERR_ARG, "sb_moe_join: dtype codes %d %d %d", h_dtype, scale_dtype, copy_dtype);
@@ -771,10 +795,10 @@ extern "C" int sb_moe_join(float* x, const float* pair_out, const int32_t* ids, 
       SB_DISPATCH_DTYPE(copy ? copy_dtype : SB_F32, TC, {
         if (vec)
           sb_launch<SB_K_ELEMENTWISE>(moe_join_kernel<4, TH, TS, TC>, grid, dim3(256), 0, stream, x, pair_out, ids, weights,
-                                      n_experts, (const TH*)h, shared, gate, gate_ld, (const TS*)scale, top, width, (TC*)copy);
+                                      weight, n_experts, (const TH*)h, shared, gate, gate_ld, (const TS*)scale, top, width, (TC*)copy);
         else
           sb_launch<SB_K_ELEMENTWISE>(moe_join_kernel<1, TH, TS, TC>, grid, dim3(256), 0, stream, x, pair_out, ids, weights,
-                                      n_experts, (const TH*)h, shared, gate, gate_ld, (const TS*)scale, top, width, (TC*)copy);
+                                      weight, n_experts, (const TH*)h, shared, gate, gate_ld, (const TS*)scale, top, width, (TC*)copy);
       });
     });
   });

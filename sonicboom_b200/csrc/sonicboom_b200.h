@@ -84,6 +84,8 @@ typedef struct SbLinearExtras {
   float gate_limit;            /* SB_EPI_SWIGLU only: > 0 makes the gated epilogue a sigmoid(gate_slope a) (b + 1), */
   float gate_slope;            /* a = min(gate, limit), b = clamp(up, -limit, limit); 0: silu(gate) * up */
   int gate_kind;               /* SB_EPI_SWIGLU only: SB_GATE_GELU_TANH makes it gelu(gate) * up; else by gate_limit */
+  const void* norm_weight2;    /* null, or a second norm of the same rows: same eps and dtypes, a weight and a */
+  void* norm_out2;             /* result of its own */
 } SbLinearExtras;
 
 /* One row's sampling record (sb_sample reads an array of them from device memory). */
@@ -112,6 +114,12 @@ int sb_rmsnorm(const float* x, const int32_t* rows, int n_rows, int width, const
 /* The same over the first `width` values of input rows that lie x_ld values apart. */
 int sb_rmsnorm_ld(const float* x, int x_ld, const int32_t* rows, int n_rows, int width, const void* weight,
                   int weight_dtype, float eps, void* out, int out_dtype, sb_stream_t stream);
+/* Two norms of the same rows with one eps: out1 with weight1, out2 with weight2 (weights of one dtype). */
+int sb_rmsnorm_pair(const float* x, int n_rows, int width, const void* weight1, const void* weight2, int weight_dtype,
+                    float eps, void* out1, void* out2, int out_dtype, sb_stream_t stream);
+/* out[t, :] = RMS norm of table[tokens[t], :] * scale, float32; an id outside the table gives NaN. */
+int sb_embed_norm(const int32_t* tokens, int n_rows, const void* table, int table_dtype, int vocab, int width,
+                  float scale, const void* weight, int weight_dtype, float eps, float* out, sb_stream_t stream);
 int sb_softcap(float* x, size_t n, float cap, sb_stream_t stream);     /* x = cap tanh(x / cap) */
 int sb_add_bias(float* x, const void* bias, int bias_dtype, int rows, int width, sb_stream_t stream);   /* x[m, n] += bias[n] */
 int sb_cast(const void* in, int in_dtype, void* out, int out_dtype, size_t n, sb_stream_t stream);
@@ -247,7 +255,7 @@ int sb_attention_plain(const void* q, void* out, int act_dtype, int n_rows, cons
  * x); the optional norm of the finished row as in sb_norm_add. */
 int sb_stream_add(const float* x, const float* add, const void* vec, int vec_dtype, int n_rows,
                   int width, float* out, const void* next_w, int next_w_dtype, float next_eps,
-                  void* normed, int normed_dtype, sb_stream_t stream);
+                  void* normed, int normed_dtype, const void* next_w2, void* normed2, sb_stream_t stream);
 /* out[r] = c0 N(z) + c1 N(z^2) + c2 N(z^3) + c3 with N(u) = u / sqrt(mean(u^2) + eps) over the row's
  * ff values, powers element by element; coef holds the four numbers. */
 int sb_polynorm(const float* z, int n_rows, int ff, const void* coef, int coef_dtype, float eps,
@@ -276,6 +284,10 @@ int sb_attn_prep(const float* proj, int n_rows, int ld, int q_off, int k_off, in
 int sb_attn_unrotate(const void* in, void* out, int dtype, int n_rows, int n_heads, int hd, int vdim,
                      int interleaved, const float* v_inv_freq, const int32_t* row_pos,
                      const float* gate, int gate_ld, sb_stream_t stream);
+/* out [rows, ld_out] from column out_off = the first vdim values of every head of in [rows, n_heads, hd], times
+ * sigmoid(gate[r * gate_ld + h * vdim + c]) (gate null: 1) and scale. */
+int sb_attn_gate(const void* in, int dtype, int n_rows, int n_heads, int hd, int vdim, const float* gate, int gate_ld,
+                 float scale, void* out, int ld_out, int out_off, sb_stream_t stream);
 /* In place on projection rows: q (at q_off) and k (at k_off), [n_heads x dim] each, are rotated
  * (the first `rot` of every head, pairs as in sb_attn_prep) and multiplied by q_scale / k_scale; z
  * [rows, n_heads * dim], if given, becomes exp(logsigmoid(z) * inv_tau).  With a2 [n_heads * dim,
@@ -297,10 +309,11 @@ int sb_linrec_scan(const float* proj, int ld, int q_off, int k_off, int v_off, c
 void sb_linrec_force_columns(int cpt);   /* 1 or 2 columns per thread in sb_linrec_scan; 0: by the sizes */
 /* out [rows, n_heads * vdim] = o / sqrt(mean over vdim of o^2 + eps) * norm_w (optional: [vdim] for
  * all heads, or [n_heads * vdim] with w_per_head) * gate(g), g at g_off of the projection row;
- * the gate is silu, or the logistic function with gate_sigmoid. */
+ * the gate is silu, or the logistic function with gate_sigmoid; times scale.  A row's results start at
+ * column out_off of a row of ld_out values. */
 int sb_linrec_out(const float* o, const float* proj, int n_rows, int ld, int g_off, int n_heads,
                   int vdim, const void* norm_w, int norm_w_dtype, int w_per_head, int gate_sigmoid,
-                  float eps, void* out, int out_dtype, sb_stream_t stream);
+                  float eps, float scale, void* out, int out_dtype, int ld_out, int out_off, sb_stream_t stream);
 
 /* ---- rows that look at their neighbours in the sequence; the layer norm ----
  * out[r] = table[tokens[r]] * scale + pair[i], i = (previous token * mul_prev + token * mul_cur) mod
@@ -349,6 +362,31 @@ int sb_delta_scan(const float* proj, int ld, int r_off, int k_off, int v_off, co
                   const int32_t* seq_row0, const int32_t* seq_slot, int n_heads, int dim, float* state,
                   float* out, sb_stream_t stream);
 
+/* ---- the gated delta rule (see gated_delta.cu) ----
+ * proj rows [q | k | v] from q_off (C = 2 n_kv_heads dim + n_heads vdim channels), a and b [n_heads] at a_off, b_off;
+ * ring [slot, taps, C] (null with one tap) and memory [slot, n_heads, vdim, dim], float32; conv_w [C, taps],
+ * a_log, dt_bias [n_heads], norm_w [vdim], float32.
+ * sb_gdelta_step: every sequence brings one row; out [rows, ld_out] from out_off = the normed, gated (silu of proj
+ * at g_off) read-out times out_scale.
+ * sb_gdelta_prep: act [rows, C] (convolved; q, k as unit vectors, q times q_scale) and the chunk matrices
+ * (sb_gdelta_mats_floats floats); sb_gdelta_scan: the recurrence over them, out [rows, n_heads, vdim], memory and
+ * ring brought up to date. */
+int sb_gdelta_step(const float* proj, int n_seqs, int ld, int q_off, int a_off, int b_off, int g_off, int n_heads,
+                   int n_kv_heads, int dim, int vdim, int taps, const float* conv_w, const float* a_log,
+                   const float* dt_bias, const int32_t* row_pos, const int32_t* seq_slot, float* ring, float* memory,
+                   float q_scale, float unit_eps, const float* norm_w, float eps, float out_scale, void* out,
+                   int out_dtype, int ld_out, int out_off, sb_stream_t stream);
+size_t sb_gdelta_mats_floats(int n_rows, int n_seqs, int n_heads);
+int sb_gdelta_prep(const float* proj, int n_rows, int ld, int q_off, int a_off, int b_off, int n_heads, int n_kv_heads,
+                   int dim, int vdim, int taps, const float* conv_w, const float* a_log, const float* dt_bias,
+                   int n_seqs, int max_new, const int32_t* seq_row0, const int32_t* seq_pos0, const int32_t* seq_slot,
+                   const float* ring, float q_scale, float unit_eps, float* act, float* mats, sb_stream_t stream);
+int sb_gdelta_scan(const float* act, const float* mats, const float* proj, int ld, int q_off, int n_heads,
+                   int n_kv_heads, int dim, int vdim, int taps, int n_seqs, const int32_t* seq_row0,
+                   const int32_t* seq_pos0, const int32_t* seq_slot, float* ring, float* memory, float* out,
+                   sb_stream_t stream);
+void sb_gdelta_force_columns(int cpt);   /* 1 or 2 columns per thread in sb_gdelta_scan; 0: by the sizes */
+
 /* ---- the state-space mixer's rows ----
  * decay [rows, n_heads] = exp(-exp(a_log) dt), dt = softplus(proj[dt_off + h] + dt_bias); the row
  * buffer's columns at xdt_off receive dt * (its columns at x_off). */
@@ -390,6 +428,10 @@ int sb_moe_max_tiles(int n_pairs, int n_experts, int tile_rows);
 /* Ids from n_experts on belong to no expert and are left out of the grouping. */
 int sb_moe_group(const int32_t* ids, int n_pairs, int n_experts, int tile_rows, int32_t* order, int32_t* meta,
                  sb_stream_t stream);
+/* The same without a router: row r's experts are table[tokens[r], 0 .. top) (int32 [vocab, top]); ids [rows, top] is
+ * written too. */
+int sb_moe_group_by_token(const int32_t* tokens, int n_rows, const int32_t* table, int vocab, int top, int n_experts,
+                          int tile_rows, int32_t* ids, int32_t* order, int32_t* meta, sb_stream_t stream);
 /* kind (SbExpert): the clamped gated form, or the square of relu (w then [experts, ff, width]). */
 int sb_moe_up(const void* a, int a_dtype, const void* w, int w_dtype, const int32_t* order,
               const int32_t* meta, int n_pairs, int n_experts, int tile_rows, int top, int ff, int width,
@@ -402,8 +444,9 @@ int sb_moe_combine(float* x, const float* pair_out, const float* weights, int n_
 
 /* x[r] += scale * (sum over the row's choices of weight * (the pair's row, or h[r] where the id is
  * n_experts or more) + sigmoid(gate[r * gate_ld]) * shared[r]); scale [width], shared, gate (without it
- * the shared row counts once) and copy (x[r] in copy_dtype) are optional. */
-int sb_moe_join(float* x, const float* pair_out, const int32_t* ids, const float* weights, int n_experts,
+ * the shared row counts once) and copy (x[r] in copy_dtype) are optional.  weights null: every choice
+ * weighs `weight`. */
+int sb_moe_join(float* x, const float* pair_out, const int32_t* ids, const float* weights, float weight, int n_experts,
                 const void* h, int h_dtype, const float* shared, const float* gate, int gate_ld,
                 const void* scale, int scale_dtype, int n_rows, int top, int width, void* copy,
                 int copy_dtype, sb_stream_t stream);

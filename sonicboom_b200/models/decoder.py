@@ -28,6 +28,7 @@ class DecoderModel:
         self.blocks = [make(BLOCKS, "block arrangement", l, dtype, device)
                        for l in spec.layers]
         self.final_norm = make(NORMS, "norm", spec.final_norm, dtype, device)
+        self.embedding_norm = make(NORMS, "norm", spec.embedding_norm, dtype, device) if spec.embedding_norm is not None else None
         # per layer: what is handed on instead of the block's own result (None: the result itself)
         self.depth_mixes = [make(DEPTH_MIXES, "depth mix", l.depth_mix, dtype, device)
                             if l.depth_mix is not None else None for l in spec.layers]
@@ -55,6 +56,8 @@ class DecoderModel:
             if m is not None:
                 req += m.tensor_requests()
         req += self.final_norm.tensor_requests()
+        if self.embedding_norm is not None:
+            req += self.embedding_norm.tensor_requests()
         if s.pair_embedding is not None:
             req.append(TensorRequest(s.pair_embedding.tensor, (s.pair_embedding.buckets + 1, s.width), "embedding"))
         if s.side_table is not None:
@@ -81,6 +84,8 @@ class DecoderModel:
             if m is not None:
                 m.bind(get)
         self.final_norm.bind(get)
+        if self.embedding_norm is not None:
+            self.embedding_norm.bind(get)
         tables = {}
         for e, inj in self.injections.items():
             if inj.tensor:
@@ -129,13 +134,19 @@ class DecoderModel:
         x = streams[0] if streams is not None else \
             torch.empty((plan.n_rows, s.width), dtype=torch.float32, device=self.device)
         ctx = StepContext(plan=plan, cache=cache, side_table=self.side_table)
-        if s.pair_embedding is None:
+        rms = self.embedding_norm.as_rms() if self.embedding_norm is not None else None
+        if s.pair_embedding is None and rms is not None:
+            ops.embed_norm(plan.tokens, self.embedding, rms[0], rms[1], x, s.embedding_scale)
+        elif s.pair_embedding is None:
             ops.embed(plan.tokens, self.embedding, x, s.embedding_scale)
         else:
             pe, prev = s.pair_embedding, ctx.model_state("prev_token")
             ops.embed_pair(plan, prev, self.embedding, self.pair_table, pe.buckets, pe.mul_prev, pe.mul_cur, x,
                            s.embedding_scale)
             ops.keep_last_token(plan, prev)
+        if self.embedding_norm is not None and (rms is None or s.pair_embedding is not None):
+            normed = self.embedding_norm.forward(x, torch.float32)
+            x = normed if streams is None else streams[0].copy_(normed)
         # an injection may add the embedding output again: it is then kept apart from the stream,
         # which blocks overwrite
         embedded = x if any(inj.embedding for inj in self.injections.values()) else None
@@ -192,13 +203,17 @@ class DecoderModel:
         out = x if x is not embedded else torch.empty_like(x)
         norm = block.input_norm()
         rms = norm.as_rms() if norm is not None else None
+        pair = norm.as_pair() if norm is not None else None
         ride = None
         if rms is not None:
             ride = (rms[0], rms[1], torch.empty(x.shape, dtype=self.dtype, device=self.device))
+        elif pair is not None:
+            normed = [torch.empty(x.shape, dtype=self.dtype, device=self.device) for _ in range(2)]
+            ride = (pair[0], pair[2], normed[0], pair[1], normed[1])
         ops.stream_add(x, embedded if inj is not None and inj.embedding else None,
                        self.injection_vectors.get(entry) if inj is not None else None, out, ride)
         if ride is not None:
-            ctx.keep_normed(norm, out, ride[2])
+            ctx.keep_normed(norm, out, ride[2] if pair is None else (ride[2], ride[4]))
         return out
 
     def _one(self):

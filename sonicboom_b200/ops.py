@@ -133,6 +133,18 @@ def add_bias(x: torch.Tensor, bias: torch.Tensor) -> torch.Tensor:
     return x
 
 
+def embed_norm(tokens: torch.Tensor, table: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor,
+               scale: float = 1.0) -> torch.Tensor:
+    """out[t] = the RMS norm (weight, eps) of table[tokens[t]] * scale, float32; an id outside the table
+    gives a row of NaN."""
+    n, width = tokens.numel(), table.shape[1]
+    assert out.dtype == torch.float32 and out.shape == (n, width) and weight.numel() == width
+    _check(lib().sb_embed_norm(_i32(tokens, "tokens"), n, _ptr(table), _code(table.dtype), table.shape[0], width,
+                               ctypes.c_float(scale), _ptr(weight), _code(weight.dtype), ctypes.c_float(eps), _ptr(out),
+                               _stream()), "embed_norm")
+    return out
+
+
 def softcap(x: torch.Tensor, cap: float) -> torch.Tensor:
     """x = cap * tanh(x / cap) in place (float32)."""
     assert x.dtype == torch.float32 and x.is_contiguous()
@@ -165,6 +177,17 @@ def rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor
     return out
 
 
+def rmsnorm_pair(x: torch.Tensor, weight1: torch.Tensor, weight2: torch.Tensor, eps: float, out1: torch.Tensor,
+                 out2: torch.Tensor) -> tuple:
+    """The RMS norms of the rows of x with two weights (of one dtype) and one eps."""
+    n, width = x.shape
+    assert x.dtype == torch.float32 and weight1.dtype == weight2.dtype and weight1.numel() == weight2.numel() == width
+    assert out1.shape == out2.shape == x.shape and out1.dtype == out2.dtype
+    _check(lib().sb_rmsnorm_pair(_ptr(x), n, width, _ptr(weight1), _ptr(weight2), _code(weight1.dtype), ctypes.c_float(eps),
+                                 _ptr(out1), _ptr(out2), _code(out1.dtype), _stream()), "rmsnorm_pair")
+    return out1, out2
+
+
 def cast(x: torch.Tensor, dtype: torch.dtype) -> torch.Tensor:
     if x.dtype == dtype:
         return x
@@ -192,7 +215,8 @@ def linear(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int = 
 
     EPI_RELU2 stores max(v, 0)^2, in every kernel.
 
-    `norm` = (weight, eps, norm_out) also writes norm_out = rmsnorm(out, weight, eps) [M,N]
+    `norm` = (weight, eps, norm_out[, weight2, norm_out2]) also writes norm_out = rmsnorm(out, weight, eps) [M,N]
+    (and norm_out2 with the second weight)
     (out must be float32): in the kernel that finishes the product where one does (the split-K
     decode form of the tcgen05 kernel), else with the norm kernel after it.
     `warm`: weights that a later kernel streams; the blocks of the tcgen05 kernel ask for them
@@ -243,16 +267,21 @@ def linear(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int = 
     fast = a.dtype == torch.bfloat16 and kernel != "plain" and K % 8 == 0
     l = lib()
     if norm is not None:
-        norm_w, norm_eps, norm_out = norm
+        norm_w, norm_eps, norm_out, norm_w2, norm_out2 = (*norm, None, None)[:5]
         assert out.dtype == torch.float32 and epilogue not in (EPI_SWIGLU, EPI_RELU2)
         assert norm_w.numel() == N and tuple(norm_out.shape) == (M, N)
+        assert norm_w2 is None or (norm_w2.numel() == N and norm_w2.dtype == norm_w.dtype
+                                   and norm_out2.shape == norm_out.shape and norm_out2.dtype == norm_out.dtype)
         fuses = fast and kernel in ("auto", "tc5") and bool(l.sb_gemm_tc5_fuses_norm(
             M, N, K, _sm_count(a.device), epilogue, _code(out.dtype), 0))
         if fuses and (kernel == "tc5" or FORCE_DECODE_KERNEL != "skinny"):
             kernel = "tc5"
         else:
             linear(a, w, out, epilogue, bias, residual, kernel, warm=warm)
-            rmsnorm(out, norm_w, norm_eps, norm_out)
+            if norm_w2 is not None:
+                rmsnorm_pair(out, norm_w, norm_w2, norm_eps, norm_out, norm_out2)
+            else:
+                rmsnorm(out, norm_w, norm_eps, norm_out)
             return out
     if kernel == "auto" and fast:
         kernel = _pick_kernel(M, N, K, a.device)
@@ -269,6 +298,8 @@ def linear(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int = 
                 extras.norm_weight, extras.norm_weight_dtype = norm_w.data_ptr(), _code(norm_w.dtype)
                 extras.norm_eps, extras.norm_out = norm_eps, norm_out.data_ptr()
                 extras.norm_out_dtype = _code(norm_out.dtype)
+                if norm_w2 is not None:
+                    extras.norm_weight2, extras.norm_out2 = norm_w2.data_ptr(), norm_out2.data_ptr()
             if warm is not None and WARM:
                 extras.warm, extras.warm_bytes = warm.data_ptr(), warm.numel() * warm.element_size()
         _check(l.sb_gemm_tc5_ex(*args[:-1], _ptr(ws), ctypes.c_size_t(ws.numel() if ws is not None else 0),
@@ -301,7 +332,8 @@ class LinearExtras(ctypes.Structure):
                 ("norm_eps", ctypes.c_float), ("norm_out", ctypes.c_void_p),
                 ("norm_out_dtype", ctypes.c_int), ("warm", ctypes.c_void_p),
                 ("warm_bytes", ctypes.c_size_t), ("rope", ctypes.POINTER(RopeStore)),
-                ("gate_limit", ctypes.c_float), ("gate_slope", ctypes.c_float), ("gate_kind", ctypes.c_int)]
+                ("gate_limit", ctypes.c_float), ("gate_slope", ctypes.c_float), ("gate_kind", ctypes.c_int),
+                ("norm_weight2", ctypes.c_void_p), ("norm_out2", ctypes.c_void_p)]
 
 
 def qkv_rope_store(h: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None, n_q_heads: int,
@@ -860,13 +892,18 @@ def mlstm_out(num: torch.Tensor, m_row: torch.Tensor, proj: torch.Tensor, n_head
 def stream_add(x: torch.Tensor, add: torch.Tensor | None, vec: torch.Tensor | None, out: torch.Tensor,
                next_norm: tuple | None = None) -> torch.Tensor:
     """out = x + add + vec row by row in float32 (`add` [rows, width] and `vec` [width] are optional;
-    out may be x).  `next_norm` = (weight, eps, normed) also writes the RMS norm of the finished rows."""
+    out may be x).  `next_norm` = (weight, eps, normed[, weight2, normed2]) also writes the RMS norm of the
+    finished rows (and a second one with another weight of the same dtype)."""
     rows, width = x.shape
     assert x.dtype == out.dtype == torch.float32 and out.shape == x.shape
     assert add is None or (add.dtype == torch.float32 and add.shape == x.shape)
     assert vec is None or vec.numel() == width
+    w2, normed2 = next_norm[3:5] if next_norm is not None and len(next_norm) > 3 else (None, None)
+    assert w2 is None or (w2.numel() == width and w2.dtype == next_norm[0].dtype
+                          and normed2.shape == next_norm[2].shape and normed2.dtype == next_norm[2].dtype)
     _check(lib().sb_stream_add(_ptr(x), _ptr(add), _ptr(vec), _code(vec.dtype) if vec is not None else 0, rows,
-                               width, _ptr(out), *_next_norm_args(next_norm, width, rows), _stream()),
+                               width, _ptr(out), *_next_norm_args(next_norm[:3] if next_norm is not None else None, width, rows),
+                               _ptr(w2), _ptr(normed2), _stream()),
            "stream_add")
     return out
 
@@ -939,6 +976,23 @@ def attn_unrotate(x: torch.Tensor, out: torch.Tensor, n_heads: int, head_size: i
     return out
 
 
+def attn_gate(x: torch.Tensor, out: torch.Tensor, n_heads: int, head_size: int, vdim: int, gate: tuple | None = None,
+              scale: float = 1.0, out_off: int = 0) -> torch.Tensor:
+    """out[:, out_off : out_off + heads * vdim] = the first vdim values of every head of x [rows, heads *
+    head_size], times `scale` and, with `gate` = (float32 rows, offset), the logistic function of each
+    value's own gate value."""
+    n = out.shape[0]
+    g_ptr, g_ld = None, 0
+    if gate is not None:
+        g, off = gate
+        assert g.dtype == torch.float32 and g.is_contiguous() and g.shape[0] == n and off + n_heads * vdim <= g.shape[1]
+        g_ptr, g_ld = g.data_ptr() + 4 * off, g.shape[1]
+    assert x.dtype == out.dtype and x.numel() == n * n_heads * head_size and out_off + n_heads * vdim <= out.shape[1]
+    _check(lib().sb_attn_gate(_ptr(x), _code(x.dtype), n, n_heads, head_size, vdim, g_ptr, g_ld, ctypes.c_float(scale),
+                              _ptr(out), out.shape[1], out_off, _stream()), "attn_gate")
+    return out
+
+
 # ---------------------------------------------------------------------- linear recurrence
 def linrec_prep(proj: torch.Tensor, q_off: int, k_off: int, n_heads: int, dim: int, q_scale: float,
                 k_scale: float, rotary_dim: int, interleaved: bool, inv_freq: torch.Tensor | None, row_pos,
@@ -993,18 +1047,19 @@ def force_linrec_columns(cpt: int) -> None:
 
 
 def linrec_out(o: torch.Tensor, proj: torch.Tensor, g_off: int, n_heads: int, vdim: int,
-               norm_w: torch.Tensor | None, eps: float, out: torch.Tensor, gate: str = "silu") -> torch.Tensor:
-    """out [rows, heads * vdim] = rms(o) per head * weight (optional: [vdim] for all heads, or
-    [heads * vdim]) * gate(g of the row); the gate is "silu" or "sigmoid"."""
+               norm_w: torch.Tensor | None, eps: float, out: torch.Tensor, gate: str = "silu",
+               scale: float = 1.0, out_off: int = 0) -> torch.Tensor:
+    """out[:, out_off : out_off + heads * vdim] = rms(o) per head * weight (optional: [vdim] for all heads, or
+    [heads * vdim]) * gate(g of the row) * scale; the gate is "silu" or "sigmoid"."""
     n, ld = proj.shape
-    assert tuple(o.shape) == (n, n_heads, vdim) and tuple(out.shape) == (n, n_heads * vdim)
+    assert tuple(o.shape) == (n, n_heads, vdim) and out.shape[0] == n and out_off + n_heads * vdim <= out.shape[1]
     assert g_off + n_heads * vdim <= ld and (norm_w is None or norm_w.numel() in (vdim, n_heads * vdim))
     assert gate in ("silu", "sigmoid")
     per_head = norm_w is not None and n_heads > 1 and norm_w.numel() == n_heads * vdim
     _check(lib().sb_linrec_out(_ptr(o), _ptr(proj), n, ld, g_off, n_heads, vdim, _ptr(norm_w),
                                _code(norm_w.dtype) if norm_w is not None else 0, 1 if per_head else 0,
-                               1 if gate == "sigmoid" else 0, ctypes.c_float(eps), _ptr(out),
-                               _code(out.dtype), _stream()), "linrec_out")
+                               1 if gate == "sigmoid" else 0, ctypes.c_float(eps), ctypes.c_float(scale), _ptr(out),
+                               _code(out.dtype), out.shape[1], out_off, _stream()), "linrec_out")
     return out
 
 
@@ -1125,6 +1180,73 @@ def delta_scan(proj: torch.Tensor, r_off: int, k_off: int, v_off: int, aux: torc
     return out
 
 
+# ---------------------------------------------------------------------- the gated delta rule
+def gated_delta(proj: torch.Tensor, q_off: int, a_off: int, b_off: int, g_off: int, plan, n_heads: int, n_kv_heads: int,
+                dim: int, vdim: int, conv_w: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor,
+                q_scale: float, unit_eps: float, norm_w: torch.Tensor, eps: float, ring: torch.Tensor | None,
+                memory: torch.Tensor, out: torch.Tensor, out_off: int = 0, scale: float = 1.0,
+                kernel: str = "auto") -> torch.Tensor:
+    """The gated delta rule over the step's projection rows (see csrc/gated_delta.cu): convolution and silu of
+    the channels [q | k | v] from q_off, unit vectors, decays from a and beta from b, the recurrence from and to
+    `memory` float32 [slot, heads, vdim, dim] and `ring` float32 [slot, taps, channels], the norm over a head's
+    outputs, the gate silu(g), times `scale`, into out[:, out_off : out_off + heads * vdim].  A step of
+    one row a sequence is one kernel; else convolution and chunk matrices, the chunked scan, norm and gate (`kernel`
+    "chunks" takes that path for any step)."""
+    n, ld = proj.shape
+    channels, taps = conv_w.shape
+    kw = n_kv_heads * dim
+    assert channels == 2 * kw + n_heads * vdim and q_off + channels <= ld and g_off + n_heads * vdim <= ld
+    assert max(a_off, b_off) + n_heads <= ld and a_log.numel() == dt_bias.numel() == n_heads and norm_w.numel() == vdim
+    for t in (proj, conv_w, a_log, dt_bias, norm_w, memory):
+        assert t.dtype == torch.float32
+    assert tuple(memory.shape[1:]) == (n_heads, vdim, dim) and out.shape[0] == n and out_off + n_heads * vdim <= out.shape[1]
+    assert taps == 1 or (ring.dtype == torch.float32 and tuple(ring.shape[1:]) == (taps, channels))
+    ring_ptr = _ptr(ring) if taps > 1 else None
+    l, c = lib(), ctypes.c_float
+    if plan.n_rows == plan.n_seqs and kernel == "auto":
+        _check(l.sb_gdelta_step(_ptr(proj), n, ld, q_off, a_off, b_off, g_off, n_heads, n_kv_heads, dim, vdim, taps,
+                                _ptr(conv_w), _ptr(a_log), _ptr(dt_bias), _i32(plan.row_pos, "row_pos"),
+                                _i32(plan.seq_slot, "seq_slot"), ring_ptr, _ptr(memory), c(q_scale), c(unit_eps),
+                                _ptr(norm_w), c(eps), c(scale), _ptr(out), _code(out.dtype), out.shape[1], out_off,
+                                _stream()), "gated_delta (one token)")
+        return out
+    act, mats = gated_delta_prep(proj, q_off, a_off, b_off, plan, n_heads, n_kv_heads, dim, vdim, conv_w, a_log, dt_bias,
+                                 q_scale, unit_eps, ring)
+    o = torch.empty((n, n_heads, vdim), dtype=torch.float32, device=proj.device)
+    gated_delta_scan(act, mats, proj, q_off, plan, n_heads, n_kv_heads, dim, vdim, taps, ring, memory, o)
+    return linrec_out(o, proj, g_off, n_heads, vdim, norm_w, eps, out, scale=scale, out_off=out_off)
+
+
+def gated_delta_prep(proj, q_off, a_off, b_off, plan, n_heads, n_kv_heads, dim, vdim, conv_w, a_log, dt_bias, q_scale,
+                     unit_eps, ring) -> tuple:
+    """(convolved rows [rows, channels] with unit q and k, chunk matrices) of `gated_delta_scan`."""
+    n, ld = proj.shape
+    channels, taps = conv_w.shape
+    act = torch.empty((n, channels), dtype=torch.float32, device=proj.device)
+    mats = torch.empty(int(lib().sb_gdelta_mats_floats(n, plan.n_seqs, n_heads)), dtype=torch.float32, device=proj.device)
+    _check(lib().sb_gdelta_prep(_ptr(proj), n, ld, q_off, a_off, b_off, n_heads, n_kv_heads, dim, vdim, taps, _ptr(conv_w),
+                                _ptr(a_log), _ptr(dt_bias), plan.n_seqs, plan.max_new, _i32(plan.seq_row0, "seq_row0"),
+                                _i32(plan.seq_pos0, "seq_pos0"), _i32(plan.seq_slot, "seq_slot"),
+                                _ptr(ring) if taps > 1 else None, ctypes.c_float(q_scale), ctypes.c_float(unit_eps),
+                                _ptr(act), _ptr(mats), _stream()), "gated_delta (chunk inputs)")
+    return act, mats
+
+
+def gated_delta_scan(act, mats, proj, q_off, plan, n_heads, n_kv_heads, dim, vdim, taps, ring, memory, o) -> torch.Tensor:
+    """o [rows, heads, vdim] = the recurrence's read-outs; `memory` and `ring` are brought up to date."""
+    _check(lib().sb_gdelta_scan(_ptr(act), _ptr(mats), _ptr(proj), proj.shape[1], q_off, n_heads, n_kv_heads, dim, vdim,
+                                taps, plan.n_seqs, _i32(plan.seq_row0, "seq_row0"), _i32(plan.seq_pos0, "seq_pos0"),
+                                _i32(plan.seq_slot, "seq_slot"), _ptr(ring) if taps > 1 else None, _ptr(memory), _ptr(o),
+                                _stream()), "gated_delta (scan)")
+    return o
+
+
+def force_gated_delta_columns(cpt: int) -> None:
+    """1 or 2: every chunked scan of the gated delta rule keeps that many columns of the state per thread where the
+    key size allows it (for measurements and tests); 0: chosen by the sizes again."""
+    lib().sb_gdelta_force_columns(int(cpt))
+
+
 # ---------------------------------------------------------------------- the state-space mixer's rows
 def ssd_prep(proj: torch.Tensor, dt_off: int, xbc: torch.Tensor, x_off: int, xdt_off: int, n_heads: int,
              vdim: int, dt_bias: torch.Tensor, a_log: torch.Tensor, decay: torch.Tensor) -> torch.Tensor:
@@ -1207,7 +1329,24 @@ def moe_route_scored(logits: torch.Tensor, correction: torch.Tensor | None, top:
 EXPERT_CLAMPED, EXPERT_RELU2 = 0, 1
 
 
-def _moe_pairs(h, ids, w_up, w_down, kind, limit, slope):
+def _moe_group_buffers(pairs, n_experts, tile, device):
+    return (torch.empty(pairs, dtype=torch.int32, device=device),
+            torch.empty(1 + 3 * int(lib().sb_moe_max_tiles(pairs, n_experts, tile)), dtype=torch.int32, device=device))
+
+
+def moe_group_by_token(tokens: torch.Tensor, table: torch.Tensor, n_experts: int, dtype, ff: int, width: int) -> tuple:
+    """The experts that `table` (int32 [vocab, top]) gives the step's tokens, and the pairs grouped by expert: (ids
+    [rows, top], order, meta) as `moe_relu2_join` takes them for experts of these sizes in this dtype."""
+    n, (vocab, top) = tokens.numel(), table.shape
+    tile = int(lib().sb_moe_tile_rows(_code(dtype), n * top, n_experts, ff, width))
+    order, meta = _moe_group_buffers(n * top, n_experts, tile, tokens.device)
+    ids = torch.empty((n, top), dtype=torch.int32, device=tokens.device)
+    _check(lib().sb_moe_group_by_token(_i32(tokens, "tokens"), n, _i32(table, "table"), vocab, top, n_experts, tile,
+                                       _ptr(ids), _ptr(order), _ptr(meta), _stream()), "moe_group_by_token")
+    return ids, order, meta
+
+
+def _moe_pairs(h, ids, w_up, w_down, kind, limit, slope, grouped=None):
     """The chosen experts applied to their rows: float32 [rows * top, width], one row per (row, choice) pair
     (left as it is where the id names no expert).  w_up is [experts, 2 (gate, up), ff, width] for
     EXPERT_CLAMPED and [experts, ff, width] for EXPERT_RELU2."""
@@ -1219,12 +1358,12 @@ def _moe_pairs(h, ids, w_up, w_down, kind, limit, slope):
     assert h.dtype == w_up.dtype == w_down.dtype
     pairs = n * top
     l = lib()
-    order = torch.empty(pairs, dtype=torch.int32, device=h.device)
     tile = int(l.sb_moe_tile_rows(_code(h.dtype), pairs, n_experts, ff, width))
-    meta = torch.empty(1 + 3 * int(l.sb_moe_max_tiles(pairs, n_experts, tile)), dtype=torch.int32, device=h.device)
+    order, meta = grouped if grouped is not None else _moe_group_buffers(pairs, n_experts, tile, h.device)
     act = torch.empty((pairs, ff), dtype=h.dtype, device=h.device)
     pair_out = torch.empty((pairs, width), dtype=torch.float32, device=h.device)
-    _check(l.sb_moe_group(_ptr(ids), pairs, n_experts, tile, _ptr(order), _ptr(meta), _stream()), "moe_group")
+    if grouped is None:
+        _check(l.sb_moe_group(_ptr(ids), pairs, n_experts, tile, _ptr(order), _ptr(meta), _stream()), "moe_group")
     _check(l.sb_moe_up(_ptr(h), _code(h.dtype), _ptr(w_up), _code(w_up.dtype), _ptr(order), _ptr(meta), pairs,
                        n_experts, tile, top, ff, width, kind, ctypes.c_float(limit), ctypes.c_float(slope), _ptr(act),
                        _stream()), "moe_up")
@@ -1245,14 +1384,16 @@ def moe_experts(h: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_up:
     return x
 
 
-def moe_relu2_join(h: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor,
+def moe_relu2_join(h: torch.Tensor, ids: torch.Tensor, weights, w_up: torch.Tensor, w_down: torch.Tensor,
                    x: torch.Tensor, shared: torch.Tensor | None = None, gate: tuple | None = None,
-                   scale: torch.Tensor | None = None, copy: torch.Tensor | None = None) -> torch.Tensor:
+                   scale: torch.Tensor | None = None, copy: torch.Tensor | None = None,
+                   grouped: tuple | None = None) -> torch.Tensor:
     """x[r] += scale * (sum over the row's choices k of weights[r, k] * y_k + sigmoid(g_r) * shared[r]), y_k
     being expert ids[r, k] applied to h[r], down (relu(up h)^2), or h[r] itself for an id from the number
     of experts on.  w_up [experts, ff, width], w_down [experts, width, ff] in h's dtype.  Optional: `shared`
     float32 rows, `gate` = (float32 rows, column) with the shared rows' g, `scale` [width], `copy`, which
-    receives the finished rows of x in its own dtype."""
+    receives the finished rows of x in its own dtype, `grouped` = (order, meta) of `moe_group_by_token`.
+    `weights` may be one number for all choices."""
     n, width = h.shape
     assert x.dtype == torch.float32 and tuple(x.shape) == (n, width)
     assert shared is None or (shared.dtype == torch.float32 and tuple(shared.shape) == (n, width))
@@ -1263,8 +1404,10 @@ def moe_relu2_join(h: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_
         g_ptr, g_ld = g.data_ptr() + 4 * col, g.shape[1]
     assert scale is None or scale.numel() == width
     assert copy is None or tuple(copy.shape) == (n, width)
-    pair_out = _moe_pairs(h, ids, w_up, w_down, EXPERT_RELU2, 0.0, 0.0)
-    _check(lib().sb_moe_join(_ptr(x), _ptr(pair_out), _ptr(ids), _ptr(weights), w_up.shape[0], _ptr(h), _code(h.dtype),
+    one = None if isinstance(weights, torch.Tensor) else float(weights)
+    pair_out = _moe_pairs(h, ids, w_up, w_down, EXPERT_RELU2, 0.0, 0.0, grouped)
+    _check(lib().sb_moe_join(_ptr(x), _ptr(pair_out), _ptr(ids), _ptr(weights) if one is None else None,
+                             ctypes.c_float(one or 0.0), w_up.shape[0], _ptr(h), _code(h.dtype),
                              _ptr(shared), g_ptr, g_ld, _ptr(scale), _code(scale.dtype) if scale is not None else 0, n,
                              ids.shape[1], width, _ptr(copy), _code(copy.dtype) if copy is not None else 0, _stream()),
            "moe_join")

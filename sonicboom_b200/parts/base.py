@@ -28,7 +28,7 @@ hint changes no result, and ignoring it costs nothing.
 """
 from __future__ import annotations
 
-from dataclasses import dataclass
+from dataclasses import dataclass, field
 from typing import Callable, Optional
 
 import torch
@@ -54,6 +54,7 @@ class StepContext:
     block_mix: Optional[tuple] = None                   # (depth mix, streams, next norm) the caller runs on that result; a block may run it with its last add
     mixed_out: Optional[torch.Tensor] = None            # what that depth mix handed on, when the block ran it
     side_table: Optional[torch.Tensor] = None           # the model's second embedding table for layers with a token input
+    kept: dict = field(default_factory=dict)            # what a part keeps for its next run in the same step (a layer may run again)
 
     def linear(self, a, w, out, epilogue, residual=None, bias=None, act_dtype=None):
         """ops.linear into float32 `out`; when `next_norm` is an RMS norm with a plain weight,
@@ -61,6 +62,13 @@ class StepContext:
         `take_normed`."""
         norm, self.next_norm, self._normed = self.next_norm, None, None
         warm, self.next_weights = self.next_weights, None
+        pair = norm.as_pair() if norm is not None else None
+        if pair is not None and out.dtype == torch.float32 and epilogue != ops.EPI_SWIGLU:
+            w1, w2, eps = pair
+            normed = tuple(torch.empty(out.shape, dtype=act_dtype or a.dtype, device=out.device) for _ in range(2))
+            ops.linear(a, w, out, epilogue, bias=bias, residual=residual, norm=(w1, eps, normed[0], w2, normed[1]), warm=warm)
+            self._normed = (norm, out, normed)
+            return out
         rms = norm.as_rms() if norm is not None else None
         if rms is None or out.dtype != torch.float32 or epilogue == ops.EPI_SWIGLU:
             return ops.linear(a, w, out, epilogue, bias=bias, residual=residual, warm=warm)
@@ -117,6 +125,11 @@ class Norm(Part):
         what a product kernel needs to apply it to its own result."""
         return None
 
+    def as_pair(self) -> Optional[tuple]:
+        """(weight1, weight2, eps) when this stands for two RMS norms of the same rows that differ in the
+        weight only (`NormPair`), else None: what a kernel needs to write both."""
+        return None
+
     def as_layer(self) -> Optional[tuple]:
         """(weight, bias or None, eps) when the norm is a layer norm, y = (x - mean) / sqrt(var + eps) *
         weight + bias, else None: what `ops.stream_join` needs to apply it to the rows it finishes."""
@@ -141,6 +154,23 @@ class Mixer(Part):
         return None
 
     def forward(self, h, ctx: StepContext, residual=None):
+        raise NotImplementedError
+
+    # A mixer that is one product, work on its rows, and one more product may open itself, so that a mixer made of
+    # several shares the two products among them: `input_matrix` / `output_matrix` (None: it does not open), and
+    #     mix_rows(proj, at, ctx, out, col, scale)
+    # which reads the input product's rows from column `at` of `proj` (float32) and writes what the output
+    # product reads, times `scale`, from column `col` of `out` (activation dtype).
+    def input_matrix(self) -> Optional[torch.Tensor]:
+        return None
+
+    def output_matrix(self) -> Optional[torch.Tensor]:
+        return None
+
+    def release_matrices(self) -> None:
+        """Called once somebody else holds the two matrices' values."""
+
+    def mix_rows(self, proj, at: int, ctx: StepContext, out, col: int = 0, scale: float = 1.0):
         raise NotImplementedError
 
     def first_weights(self, rows: int) -> Optional[torch.Tensor]:

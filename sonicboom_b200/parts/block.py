@@ -209,7 +209,12 @@ class ParallelResidualBlock(Block):
     """One norm feeds both sublayers: h = norm(x); x <- x + mix(h) + ffn(h) (without a feed-forward,
     x + mix(h)).  The mixer adds its result to the stream in its last product, the feed-forward
     adds its own to that, so the sum is ((x + mix) + ffn) in float32; the norm that comes after the
-    block can ride on the last of the two products."""
+    block can ride on the last of the two products.
+
+    With a `feed_forward_norm` in the spec each sublayer has a norm of its own on the same x: x <- x +
+    mix(norm1(x)) + ffn(norm2(x)).  Both norms are one reading of the row (`NormPair`).  The feed-forward then
+    adds its result first: a mixer always ends in a product, which the next block's norms ride on, a mixture of
+    experts does not."""
 
     def __init__(self, spec, dtype, device):
         self.dtype = dtype
@@ -218,6 +223,12 @@ class ParallelResidualBlock(Block):
         self.feed_forward = make(FEED_FORWARDS, "feed-forward", spec.feed_forward, dtype, device) \
             if spec.feed_forward is not None else None
         self.parts = [self.mixer_norm, self.mixer] + ([self.feed_forward] if self.feed_forward is not None else [])
+        self.pair = None
+        if self.feed_forward is not None and spec.feed_forward_norm is not None:
+            from .norm import NormPair
+            norm2 = make(NORMS, "norm", spec.feed_forward_norm, dtype, device)
+            self.parts.append(norm2)
+            self.pair = NormPair(self.mixer_norm, norm2)
 
     def tensor_requests(self):
         return [r for p in self.parts for r in p.tensor_requests()]
@@ -233,16 +244,23 @@ class ParallelResidualBlock(Block):
         return self.mixer.state_need()
 
     def input_norm(self):
-        return self.mixer_norm
+        return self.mixer_norm if self.pair is None else self.pair
 
     def first_weights(self, rows):
-        return self.mixer.first_weights(rows)
+        return self.mixer.first_weights(rows) if self.pair is None else None
 
     def forward(self, x, ctx):
         after, after_weights = ctx.after_block_norm, ctx.after_block_weights
-        h = ctx.take_normed(self.mixer_norm, x)
+        norm = self.input_norm()
+        h = ctx.take_normed(norm, x)
         if h is None:
-            h = self.mixer_norm.forward(x, self.dtype)
+            h = norm.forward(x, self.dtype)
+        if self.pair is not None:
+            h, f = h
+            ctx.next_norm = ctx.next_weights = None
+            x = self.feed_forward.forward(f, ctx, residual=x)
+            ctx.next_norm, ctx.next_weights = after, after_weights
+            return self.mixer.forward(h, ctx, residual=x)
         if self.feed_forward is None:
             ctx.next_norm, ctx.next_weights = after, after_weights
             return self.mixer.forward(h, ctx, residual=x)

@@ -28,8 +28,8 @@ def interleave_gate_up(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
 class SwiGLU(FeedForward):
     """y = Wdown (act(Wgate f) * (Wup f)).  `activation` is "silu" or "gelu_tanh" (gelu in its tanh
     form, 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))); `params` may give `names`, the tensor
-    names of the three matrices after the prefix.  With silu the product's epilogue applies the
-    activation; with gelu_tanh the product's float32 rows go through the activation kernel."""
+    names of the three matrices after the prefix.  The product's epilogue applies the activation; an intermediate
+    size that is no multiple of `ops.SWIGLU_BLOCK` goes through the activation kernel."""
 
     def __init__(self, spec, dtype, device):
         from ..config.specs import ConfigError
@@ -37,9 +37,6 @@ class SwiGLU(FeedForward):
         if spec.activation not in ("silu", "gelu_tanh"):
             raise ConfigError(f"feed-forward activation {spec.activation!r} is not built (silu, gelu_tanh)")
         self.interleaved = spec.intermediate % ops.SWIGLU_BLOCK == 0
-        if not self.interleaved and spec.activation == "silu":
-            raise ConfigError(f"intermediate_size {spec.intermediate} must be a multiple of "
-                              f"{ops.SWIGLU_BLOCK} for the fused gate/up product")
         self.names = tuple(dict(spec.params).get("names", ("gate_proj.weight", "up_proj.weight", "down_proj.weight")))
         self.w_gate_up = self.w_down = None
 
@@ -60,7 +57,7 @@ class SwiGLU(FeedForward):
     def forward(self, h, ctx, residual=None):
         rows, ff = h.shape[0], self.spec.intermediate
         t = torch.empty((rows, ff), dtype=self.dtype, device=h.device)
-        if self.spec.activation == "silu":
+        if self.spec.activation == "silu" and self.interleaved:
             ops.linear(h, self.w_gate_up, t, ops.EPI_SWIGLU)
         elif self.interleaved:
             ops.linear(h, self.w_gate_up, t, ops.EPI_SWIGLU, gate_kind=ops.GATE_KINDS[self.spec.activation])
@@ -208,6 +205,10 @@ class ExpertsSquaredRelu(FeedForward):
     the prefix: router [experts + identity, width], the correction [experts + identity], e<j>.up
     [intermediate, width], e<j>.down [width, intermediate]; the shared gate's [1, width].
 
+    With `by_token` = (table name, vocab) there is no router: an integer table [vocab, top] names every token id's
+    experts, each weighted 1 / top (no identities, no correction).  A step's grouping is then made from the
+    tokens alone, once for all runs of the layer in the step.
+
     The shared gate's row rides on the router product.  Grouping and tiles are those of
     `experts_glu_clamped`; the last kernel (`ops.moe_relu2_join`) adds the choices, identities and the gated
     shared expert and joins the stream, so a block calls `join` rather than `forward`."""
@@ -222,6 +223,9 @@ class ExpertsSquaredRelu(FeedForward):
             raise ConfigError(f"a mixture of {self.n_experts} experts and {self.identity} identities cannot choose {self.top}")
         self.scale, self.correction_name = float(p.get("scale", 1.0)), p.get("correction", "correction")
         shared, self.gate_name = p.get("shared"), p.get("shared_gate")
+        self.by_token, self.table = p.get("by_token"), None
+        if self.by_token and (self.identity or self.gate_name):
+            raise ConfigError("experts chosen by token id go without identity outputs and without a shared gate")
         self.shared = make(FEED_FORWARDS, "feed-forward", shared, dtype, device) if shared is not None else None
         if self.shared is None:
             self.gate_name = None
@@ -229,7 +233,10 @@ class ExpertsSquaredRelu(FeedForward):
 
     def tensor_requests(self):
         p, d, ff = self.spec.prefix, self.spec.width, self.spec.intermediate
-        req = [TensorRequest(p + "router", (self.outputs, d)), TensorRequest(p + self.correction_name, (self.outputs,), "bias")]
+        if self.by_token:
+            req = [TensorRequest(p + self.by_token[0], (int(self.by_token[1]), self.top), "table", below=self.n_experts)]
+        else:
+            req = [TensorRequest(p + "router", (self.outputs, d)), TensorRequest(p + self.correction_name, (self.outputs,), "bias")]
         for j in range(self.n_experts):
             req += [TensorRequest(f"{p}e{j}.up", (ff, d)), TensorRequest(f"{p}e{j}.down", (d, ff))]
         if self.gate_name:
@@ -238,11 +245,13 @@ class ExpertsSquaredRelu(FeedForward):
 
     def bind(self, get):
         p = self.spec.prefix
-        router = [get(p + "router")] + ([get(p + self.gate_name)] if self.gate_name else [])
-        if len({t.dtype for t in router}) > 1:
-            router = [t.float() for t in router]
-        self.w_router = torch.cat(router).contiguous()
-        self.correction = get(p + self.correction_name).float().contiguous()
+        if self.by_token:
+            from ..config.specs import ConfigError
+            self.table = get(p + self.by_token[0])
+            if self.table.numel() and not 0 <= int(self.table.min()) <= int(self.table.max()) < self.n_experts:
+                raise ConfigError(f"{p}{self.by_token[0]} names an expert outside 0 .. {self.n_experts - 1}")
+        else:
+            self._bind_router(get)
         ups = [get(f"{p}e{j}.up") for j in range(self.n_experts)]
         downs = [get(f"{p}e{j}.down") for j in range(self.n_experts)]
         if len({t.dtype for t in ups + downs}) > 1:
@@ -251,10 +260,27 @@ class ExpertsSquaredRelu(FeedForward):
         if self.shared is not None:
             self.shared.bind(get)
 
+    def _bind_router(self, get):
+        p = self.spec.prefix
+        router = [get(p + "router")] + ([get(p + self.gate_name)] if self.gate_name else [])
+        if len({t.dtype for t in router}) > 1:
+            router = [t.float() for t in router]
+        self.w_router = torch.cat(router).contiguous()
+        self.correction = get(p + self.correction_name).float().contiguous()
+
     def join(self, h, ctx, x, scale=None, copy=None):
         """x += scale * (the mixture of h), in place; `copy` receives the finished rows in its dtype."""
         rows = h.shape[0]
         ctx.next_norm = ctx.next_weights = None      # the last kernel is not a product: nothing rides on one
+        if self.by_token:
+            if self not in ctx.kept:
+                ctx.kept[self] = ops.moe_group_by_token(ctx.plan.tokens, self.table, self.n_experts, self.w_up.dtype,
+                                                        self.spec.intermediate, self.spec.width)
+            ids, *grouped = ctx.kept[self]
+            shared = self.shared.forward(h, ctx) if self.shared is not None else None
+            a = h if h.dtype == self.w_up.dtype else ops.cast(h, self.w_up.dtype)
+            return ops.moe_relu2_join(a, ids, 1.0 / self.top, self.w_up, self.w_down, x, shared=shared, scale=scale, copy=copy,
+                                      grouped=grouped)
         logits = torch.empty((rows, self.w_router.shape[0]), dtype=torch.float32, device=h.device)
         ids = torch.empty((rows, self.top), dtype=torch.int32, device=h.device)
         weights = torch.empty((rows, self.top), dtype=torch.float32, device=h.device)

@@ -88,6 +88,28 @@ class LayerNorm(Norm):
         return ops.layernorm(x, self.weight, self.eps, out, rows, bias=self.bias)
 
 
+class NormPair(Norm):
+    """Two RMS norms of the same rows: what a block whose sublayers have norms of their own on one input names as its
+    `input_norm()`.  `forward` returns both results; with one eps (and weights of one dtype) a kernel writes
+    both from one reading of the row, here or where the rows are finished (`as_pair`)."""
+
+    def __init__(self, first, second):
+        self.first, self.second = first, second
+
+    def as_pair(self):
+        a, b = self.first.as_rms(), self.second.as_rms()
+        if a is None or b is None or a[1] != b[1] or a[0].dtype != b[0].dtype:
+            return None
+        return a[0], b[0], a[1]
+
+    def forward(self, x, out_dtype, rows=None):
+        pair = self.as_pair() if rows is None else None
+        if pair is None:
+            return self.first.forward(x, out_dtype, rows), self.second.forward(x, out_dtype, rows)
+        return ops.rmsnorm_pair(x, pair[0], pair[1], pair[2], torch.empty(x.shape, dtype=out_dtype, device=x.device),
+                                torch.empty(x.shape, dtype=out_dtype, device=x.device))
+
+
 class StreamCast(Norm):
     """Not a norm: the rows as they are, in the dtype asked for.  A block whose sublayers read the
     stream itself names this as its `input_norm()`, so that whatever finishes the stream's rows

@@ -22,6 +22,8 @@ that attention layers of newer designs combine:
 * `softcap` = c: a score s becomes c tanh(s / c) before the softmax;
 * `gate` = name: a matrix [heads, width]; head h's result is multiplied by the logistic function
   of its product with the mixer's input (it rides on the input product);
+* `value_gate` = name: a matrix [heads*vdim, width]; every value of the concatenated heads is multiplied by the
+  logistic function of its own product with the mixer's input (it rides on the input product too);
 * `conv` = taps: every channel of q, k and v passes a short causal convolution over time right after the
   projection (tensors: the projection's name + ".conv", [channels, taps]); the last taps - 1 projected
   values of a sequence are state of the cache;
@@ -38,7 +40,8 @@ Tensors after the prefix: q [heads*head_dim, width], k [kv_heads*head_dim, width
 name.  All input projections are one product; `ops.attn_prep` finishes its float32 rows into
 queries and cache rows (`ops.conv_heads` with a convolution and nothing else to do to the heads), the
 framework's attention kernels run on them unchanged, and
-`ops.attn_unrotate` turns results back and drops the padding where either is needed."""
+`ops.attn_unrotate` turns results back and drops the padding where either is needed (`ops.attn_gate` with a
+`value_gate`, or as one side of a mixer that shares its products)."""
 from __future__ import annotations
 
 import math
@@ -89,6 +92,10 @@ class WindowAttention(Mixer):
         self.rotate_values = bool(p.get("rotate_values", False))
         self.qk_norm, self.sink_name = p.get("qk_norm"), p.get("sink")
         self.bias_names, self.gate_name = p.get("bias"), p.get("gate")
+        self.value_gate = p.get("value_gate")
+        if self.value_gate and (self.gate_name or self.rotate_values):
+            raise ConfigError("a gate for every value goes with unrotated values and no gate per head")
+        self.gate_name = self.value_gate or self.gate_name
         self.softcap = float(p.get("softcap", 0.0) or 0.0)
         self.taps, self.chunk = int(p.get("conv", 0) or 0), int(p.get("chunk", 0) or 0)
         self.distance_bias = p.get("distance_bias")
@@ -128,7 +135,7 @@ class WindowAttention(Mixer):
                 self.v_inv_freq = frequency_table(spec.position.theta, self.vdim, device)
         self.qw, self.kw = self.hq * self.dim, self.hkv * self.dim
         self.vw = 0 if self.values_are_keys else self.hkv * self.vdim
-        self.gw = self.hq if self.gate_name else 0
+        self.gw = 0 if not self.gate_name else self.hq * self.vdim if self.value_gate else self.hq
         if self.bias_names and self.values_are_keys:
             raise ConfigError("biases of q, k and v need a value projection of its own")
         if self.taps and (self.values_are_keys or self.gate_name):
@@ -157,7 +164,7 @@ class WindowAttention(Mixer):
         if self.bias_names:
             req += [TensorRequest(p + n, (w,), "bias") for n, w in zip(self.bias_names, (self.qw, self.kw, self.vw))]
         if self.gate_name:
-            req.append(TensorRequest(p + self.gate_name, (self.hq, d)))
+            req.append(TensorRequest(p + self.gate_name, (self.gw, d)))
         if self.sink_name:
             req.append(TensorRequest(p + self.sink_name, (self.hq,), "bias"))
         if self.taps:
@@ -196,18 +203,57 @@ class WindowAttention(Mixer):
         late = self.w_in.dtype == torch.bfloat16 and ops.requests_weights_late(rows, n, k, self.w_in.device)
         return self.w_in if late else None
 
+    def input_matrix(self):
+        """Opens only without what belongs to the whole product's rows (biases, convolutions)."""
+        return None if self.taps or self.bias_names else self.w_in
+
+    def output_matrix(self):
+        return self.w_o
+
+    def release_matrices(self):
+        self.w_in = self.w_o = None
+
+    def mix_rows(self, proj, at, ctx, out, col=0, scale=1.0):
+        mixed = self._attend(proj, at, ctx)
+        if self.rotate_values or (self.gw and not self.value_gate):
+            mixed = self._finish(mixed, proj, at, ctx)
+            return ops.attn_gate(mixed, out, self.hq, self.vdim, self.vdim, None, scale, col)
+        return ops.attn_gate(mixed, out, self.hq, self.hd, self.vdim, (proj, at + self.qw) if self.value_gate else None,
+                             scale, col)
+
     def forward(self, h, ctx, residual=None):
-        rows, plan = h.shape[0], ctx.plan
-        k_off = self.qw + self.gw
-        width_in = k_off + ((self.kw + self.vw) if ctx.owns_cache else 0)
-        storage = ctx.kv_storage()
-        g = plan.groups[ctx.kv_group()]
+        rows = h.shape[0]
+        width_in = self.qw + self.gw + ((self.kw + self.vw) if ctx.owns_cache else 0)
         proj = torch.empty((rows, width_in), dtype=torch.float32, device=h.device)
         if self.b_in is not None:
             ops.linear(h, self.w_in[:width_in], proj, ops.EPI_BIAS, bias=self.b_in[:width_in])
         else:
             ops.linear(h, self.w_in[:width_in], proj)
-        q = torch.empty((rows, self.hq, self.hd), dtype=self.dtype, device=h.device)
+        mixed = self._attend(proj, 0, ctx)
+        if self.value_gate:
+            gated = torch.empty((rows, self.hq * self.vdim), dtype=self.dtype, device=h.device)
+            mixed = ops.attn_gate(mixed, gated, self.hq, self.hd, self.vdim, (proj, self.qw))
+        elif self.rotate_values or self.hd != self.vdim or self.gw:
+            mixed = self._finish(mixed, proj, 0, ctx)
+        out = residual if residual is not None else \
+            torch.empty((rows, self.spec.width), dtype=torch.float32, device=h.device)
+        return ctx.linear(mixed, self.w_o, out, ops.EPI_RESIDUAL if residual is not None else ops.EPI_NONE,
+                          residual=residual, act_dtype=self.dtype)
+
+    def _finish(self, mixed, proj, at, ctx):
+        """The heads' results turned back, without padding, times their gates (one number per head)."""
+        rows = proj.shape[0]
+        turned = torch.empty((rows, self.hq * self.vdim), dtype=self.dtype, device=proj.device)
+        return ops.attn_unrotate(mixed, turned, self.hq, self.hd, self.vdim, self.interleaved, self.v_inv_freq,
+                                 ctx.plan.row_pos, gate=(proj, at + self.qw) if self.gw else None)
+
+    def _attend(self, proj, at, ctx):
+        """The heads' results [rows, heads * hd] from the input product's rows, which start at column `at`."""
+        rows, plan = proj.shape[0], ctx.plan
+        k_off, width_in = at + self.qw + self.gw, proj.shape[1]
+        storage = ctx.kv_storage()
+        g = plan.groups[ctx.kv_group()]
+        q = torch.empty((rows, self.hq, self.hd), dtype=self.dtype, device=proj.device)
         if self.taps and not ctx.owns_cache:
             from ..config.specs import ConfigError
             raise ConfigError("attention with convolved projections has keys and values of its own")
@@ -219,20 +265,12 @@ class WindowAttention(Mixer):
             if self.taps:
                 turned = torch.empty_like(proj)
                 proj = ops.causal_conv(proj, 0, width_in, self.w_conv, None, plan, state, turned)
-            ops.attn_prep(proj, 0, k_off, -1 if self.values_are_keys else k_off + self.kw, self.hq, self.hkv,
+            ops.attn_prep(proj, at, k_off, -1 if self.values_are_keys else k_off + self.kw, self.hq, self.hkv,
                           self.dim, self.vdim, self.hd, self.rot, self.interleaved, self.inv_freq, self.v_inv_freq,
                           self.q_norm, self.k_norm, self.eps, plan.row_seq, plan.row_pos, g.page_off, g.page_ids,
                           g.page_size, storage if ctx.owns_cache else None, q, head_norm=self.head_norm,
                           rot_scale=self.rot_scale)
-        mixed = torch.empty((rows, self.hq * self.hd), dtype=self.dtype, device=h.device)
-        ops.attention(q, mixed, plan, ctx.kv_group(), storage, self.hq, self.hkv, self.hd, self.spec.window,
-                      self.spec.scale, warm=self.w_o, sink=self.sink, softcap=self.softcap, chunk=self.chunk,
-                      bias=self.bias)
-        if self.rotate_values or self.hd != self.vdim or self.gw:
-            turned = torch.empty((rows, self.hq * self.vdim), dtype=self.dtype, device=h.device)
-            mixed = ops.attn_unrotate(mixed, turned, self.hq, self.hd, self.vdim, self.interleaved,
-                                      self.v_inv_freq, plan.row_pos, gate=(proj, self.qw) if self.gw else None)
-        out = residual if residual is not None else \
-            torch.empty((rows, self.spec.width), dtype=torch.float32, device=h.device)
-        return ctx.linear(mixed, self.w_o, out, ops.EPI_RESIDUAL if residual is not None else ops.EPI_NONE,
-                          residual=residual, act_dtype=self.dtype)
+        mixed = torch.empty((rows, self.hq * self.hd), dtype=self.dtype, device=proj.device)
+        return ops.attention(q, mixed, plan, ctx.kv_group(), storage, self.hq, self.hkv, self.hd, self.spec.window,
+                             self.spec.scale, warm=self.w_o, sink=self.sink, softcap=self.softcap, chunk=self.chunk,
+                             bias=self.bias)

@@ -19,6 +19,7 @@ class TensorRequest:
     shape: tuple                # -1: any size there
     role: str = "matrix"        # matrix | embedding | bias | norm | table (integers)
     optional: bool = False      # absent is fine, present is not "unexpected"
+    below: int = 0              # a table's integers are below this (for random ones; the entries of a row then differ)
 
 
 class WeightError(ValueError):

@@ -125,7 +125,7 @@ class RandomSource:
     def tensor(self, name) -> torch.Tensor:
         r = self.requests[name]
         if r.role == "table":
-            return torch.zeros(r.shape, dtype=torch.int32, device=self.device)
+            return self._table(r).to(self.device)
         mean, std = {"norm": (1.0, self.norm_std), "bias": (0.0, self.bias_std)}.get(
             r.role, (0.0, self.std))
         key0, key1 = tensor_key(self.seed, name)
@@ -137,6 +137,21 @@ class RandomSource:
                 return ops.random_normal(out, key0, key1, mean, std)
         x = torch.from_numpy(normal_numpy(n, key0, key1, mean, std)).reshape(r.shape)
         return x.to(self.dtype)
+
+
+    def _table(self, r) -> torch.Tensor:
+        """Integers below `r.below` (zeros without it), the entries of a row all different: row i steps from a
+        random start by a random stride that cannot meet itself within the row."""
+        if r.below <= 0:
+            return torch.zeros(r.shape, dtype=torch.int32)
+        cols = r.shape[-1] if r.shape else 1
+        if cols > r.below:
+            raise ValueError(f"{r.name}: {cols} different integers below {r.below}")
+        rows = int(np.prod(r.shape[:-1], dtype=np.int64))
+        w = _philox(np.arange(rows, dtype=np.uint64), *tensor_key(self.seed, r.name))
+        start, stride = w[0] % np.uint64(r.below), np.uint64(1) + w[1] % np.uint64(r.below // cols)
+        t = (start[:, None] + stride[:, None] * np.arange(cols, dtype=np.uint64)) % np.uint64(r.below)
+        return torch.from_numpy(t.astype(np.int32)).reshape(r.shape)
 
 
 def write_random_model(model_dir, config_dict: dict, seed: int, std=0.02, bias_std=None,
