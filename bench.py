@@ -1341,7 +1341,7 @@ def debisun_kernels(bench, z, rows, context):
     from sonicboom_b200.ops import _check, _code, _ptr, _stream, lib
     pair_out = torch.randn(pairs, W, device=dev)
     rec("moe_join: choices, identities, gated shared expert, scale, copy", timed(lambda: _check(lib().sb_moe_join(
-        _ptr(x), _ptr(pair_out), _ptr(ids), _ptr(wts), E, _ptr(h), _code(bf), _ptr(y), _ptr(logits), E + I + 1, _ptr(wb), _code(bf),
+        _ptr(x), _ptr(pair_out), _ptr(ids), _ptr(wts), 0.0, E, _ptr(h), _code(bf), _ptr(y), _ptr(logits), E + I + 1, _ptr(wb), _code(bf),
         rows, top, W, _ptr(nb), _code(bf), _stream()), "moe_join")), pairs * W * 4 + rows * W * 16)
     rec("like: moe_combine", timed(lambda: _check(lib().sb_moe_combine(_ptr(x), _ptr(pair_out), _ptr(wts), rows, top, W, _stream()),
                                                   "moe_combine")), pairs * W * 4 + rows * W * 8)
