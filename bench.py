@@ -8,6 +8,7 @@ sizes of Qwen2.5-7B with random weights on one B200.
     python bench.py --arch leguvik [--sizes w2048,w3584] [--prompt 2048] [--batch 8] [--steps K]
     python bench.py --arch bulodra [--sizes w2048,w3584] [--prompt 2048] [--batch 8] [--steps K]
     python bench.py --arch debisun [--sizes w2048,w3584] [--prompt 2048] [--batch 8] [--steps K]
+    python bench.py --arch sipilorn [--sizes w2048,w3584] [--prompt 2048] [--batch 8] [--steps K]
 
 Prints ONE JSON line.  (`--arch zolulix` is a measurement of its own: the Zolulix design beside the
 Qwen2.5 decoder of equal sizes and its kernels alone; without it the workload below runs.)  A "step" is one decode step of the whole batch.  The default run is a
@@ -1402,6 +1403,236 @@ def run_debisun(args) -> int:
     return 0
 
 
+# ---------------------------------------------------------------------------- --arch sipilorn
+def sipilorn_config(width, n_layers, vocab, heads, kv_heads, dim, window, d_heads, d_kv, d_dim, d_vdim, p_heads, p_kv, taps, ff,
+                    experts=0, top=0, expert_ff=0):
+    """A Sipilorn model of the given layer sizes: three delta layers and a parallel one in turn, every layer with a
+    dense feed-forward, or (with `experts`) every second one with experts by token id; no loop."""
+    delta = {"heads": d_heads, "kv_heads": d_kv, "dim": d_dim, "vdim": d_vdim, "conv": taps}
+    left = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "mask": {"size": window},
+            "rot": {"base": 200000.0, "dims": dim // 2}}
+    right = dict(delta, heads=p_heads, kv_heads=p_kv)
+    dense = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": expert_ff}}
+    layers = [{"type": "delta", "mixer": delta} if i % 4 < 3 else
+              {"type": "parallel", "mixer": {"left": left, "right": right, "left_scale": 0.9, "right_scale": 0.7}} for i in range(n_layers)]
+    for i, L in enumerate(layers):
+        L["mlp"] = moe if experts and i % 2 else dense
+    return {"architecture": "Sipilorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "logit_softcap": 30.0, "layers": layers}
+
+
+def sipilorn_mefupel_config(z):
+    """The Mefupel model beside it: three gated-linear-attention layers and a parallel one in turn, with states,
+    projections, windows and feed-forward values of the same sizes (a recurrence head per key head, values as wide
+    as all of its heads')."""
+    m = mefupel_config(width=z["width"], n_layers=1, ff=z["ff"], vocab=z["vocab"], heads=z["heads"], kv_heads=z["kv_heads"], dim=z["dim"],
+                       window=z["window"], r_heads=1, r_dim=z["d_dim"], r_vdim=z["d_vdim"])
+    gla = {"heads": z["d_kv"], "dim": z["d_dim"], "vdim": z["d_vdim"] * z["d_heads"] // z["d_kv"], "tau": 12.0, "decay_rank": 16}
+    left = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["dim"], "scale": z["dim"] ** -0.5,
+            "mask": {"size": z["window"]}, "rot": {"base": 20000.0, "dims": z["dim"] // 2}}
+    right = {"heads": z["p_kv"], "dim": z["d_dim"], "vdim": z["d_vdim"] * z["p_heads"] // z["p_kv"],
+             "rot": {"base": 100000.0, "dims": z["d_dim"]}, "decay": [0.9 + 0.099 * (i + 1) / z["p_kv"] for i in range(z["p_kv"])]}
+    m["layers"] = [{"type": "gla", "mixer": gla} if i % 4 < 3 else {"type": "parallel", "mixer": {"left": left, "right": right}}
+                   for i in range(z["n_layers"])]
+    for L in m["layers"]:
+        L["mlp"] = {"kind": "dense", "ff": z["ff"]}
+    return m
+
+
+SIPILORN_SIZES = {
+    # Mefupel is the closest design (mixer and feed-forward side by side, recurrences with a matrix state, windowed attention
+    # beside one); its dense feed-forward has two matrices for Sipilorn's three
+    "w2048": dict(width=2048, n_layers=8, vocab=32768, heads=16, kv_heads=4, dim=128, window=1024, d_heads=32, d_kv=16, d_dim=128,
+                  d_vdim=128, p_heads=16, p_kv=8, taps=4, ff=8192),
+    "w3584": dict(width=3584, n_layers=8, vocab=32768, heads=28, kv_heads=4, dim=128, window=4096, d_heads=56, d_kv=28, d_dim=128,
+                  d_vdim=128, p_heads=28, p_kv=14, taps=4, ff=18944),
+}
+SIPILORN_EXPERTS = {"w2048": dict(experts=32, top=4, expert_ff=1024), "w3584": dict(experts=64, top=6, expert_ff=1536)}
+
+
+def sipilorn_kernels(bench, z, moe, rows, context):
+    """Each kernel that came with Sipilorn (or was extended for it) alone at `rows` rows (one sequence of `rows`
+    tokens when rows > 64, else `rows` sequences that hold `context` tokens each and go on by one), with the bytes it
+    must read and write once, and beside each the like kernel of the framework's other models at the same sizes."""
+    import torch
+    from sonicboom_b200 import ops
+    from sonicboom_b200.cache.kv import Cache, KVNeed, StateNeed
+    from sonicboom_b200.engine.step import StepEntry, StepPlan
+    from sonicboom_b200.parts.rotary import frequency_table
+    dev, pk, timed = bench.dev, bench.pk, bench.timed
+    W, bf = z["width"], torch.bfloat16
+    out = {}
+
+    def rec(name, ms, nbytes, flops=0):
+        out[name] = {"us": round(ms * 1e3, 2), "bytes": int(nbytes),
+                     "hbm_frac": round(nbytes / (ms / 1e3) / 1e9 / pk["hbm_gbs"], 3)}
+        if flops:
+            out[name]["tflops"] = round(flops / (ms / 1e3) / 1e12, 2)
+    prompt = rows > 64
+    n_seqs, new = (1, rows) if prompt else (rows, 1)
+    past = 0 if prompt else context
+    H, G, d, dv, taps = z["d_heads"], z["d_kv"], z["d_dim"], z["d_vdim"], z["taps"]
+    aH, aG, ad, win = z["heads"], z["kv_heads"], z["dim"], z["window"]
+    kw, C = G * d, 2 * G * d + H * dv
+    hk = H * d
+    needs = {"ring": StateNeed((taps, C)), "memory": StateNeed((H, dv, d)), "shift": StateNeed((taps - 1, C))}
+    cache = Cache([KVNeed(aG, ad, win)], [needs], n_seqs * (past + new + 64), bf, dev, n_slots=n_seqs)
+    slots = [cache.open() for _ in range(n_seqs)]
+    for s in slots:
+        if past:
+            cache.reserve(s, past)
+            cache.advance(s, past)
+        cache.reserve(s, past + new)
+    plan = StepPlan(cache, [StepEntry(s, [0] * new, []) for s in slots], dev)
+    kind = f"{n_seqs} sequence(s) of {new}" + (f" after {past}" if past else "")
+    # rows of the stream
+    x, vec = torch.randn(rows, W, device=dev), torch.randn(W, device=dev).to(bf)
+    wb, xo = torch.ones(W, device=dev, dtype=bf), torch.empty(rows, W, device=dev)
+    n1, n2 = torch.empty(rows, W, device=dev, dtype=bf), torch.empty(rows, W, device=dev, dtype=bf)
+    rec("rmsnorm_pair", timed(lambda: ops.rmsnorm_pair(x, wb, wb, 1e-5, n1, n2)), rows * W * 8)
+    rec("like: rmsnorm", timed(lambda: ops.rmsnorm(x, wb, 1e-5, n1)), rows * W * 6)
+    rec("stream_add + two norms", timed(lambda: ops.stream_add(x, None, vec, xo, (wb, 1e-5, n1, wb, n2))), rows * W * 12)
+    rec("like: stream_add + norm", timed(lambda: ops.stream_add(x, None, vec, xo, (wb, 1e-5, n1))), rows * W * 10)
+    table = torch.randn(z["vocab"], W, device=dev).to(bf)
+    toks = torch.randint(0, z["vocab"], (rows,), generator=bench.gen).int().to(dev)
+    rec("embed_norm", timed(lambda: ops.embed_norm(toks, table, wb, 1e-5, xo)), rows * W * 6)
+    rec("like: embed", timed(lambda: ops.embed(toks, table, xo)), rows * W * 6)
+    # the gated delta rule
+    g_off = C
+    b_off = g_off + H * dv
+    a_off = b_off + H
+    proj = torch.randn(rows, (a_off + H + 3) // 4 * 4, device=dev)
+    conv_w = torch.randn(C, taps, device=dev)
+    a_log, dt, norm_w = torch.zeros(H, device=dev), torch.zeros(H, device=dev), torch.ones(dv, device=dev)
+    ring, memory = cache.state[(0, "ring")], cache.state[(0, "memory")]
+    mixed = torch.empty(rows, H * dv, device=dev, dtype=bf)
+    o = torch.empty(rows, H, dv, device=dev)
+    state_bytes, ring_bytes = n_seqs * H * d * dv * 8, n_seqs * taps * C * 4
+    delta_flops, lin_flops = 7 * rows * H * d * dv, 5 * rows * H * d * dv
+    if prompt:
+        act, mats = ops.gated_delta_prep(proj, 0, a_off, b_off, plan, H, G, d, dv, conv_w, a_log, dt, d ** -0.5, 1e-6, ring)
+        rec("gated delta: convolution, unit vectors, chunk matrices",
+            timed(lambda: ops.gated_delta_prep(proj, 0, a_off, b_off, plan, H, G, d, dv, conv_w, a_log, dt, d ** -0.5, 1e-6, ring)),
+            rows * C * 8 + mats.numel() * 4)
+        for cpt in (1, 2):
+            ops.force_gated_delta_columns(cpt)
+            rec(f"gated delta: chunked scan, {cpt} column(s) a thread ({kind}; {H} heads of {d} x {dv})",
+                timed(lambda: ops.gated_delta_scan(act, mats, proj, 0, plan, H, G, d, dv, taps, ring, memory, o)),
+                rows * (C + H * dv) * 4 + mats.numel() * 4 + state_bytes, delta_flops)
+        ops.force_gated_delta_columns(0)
+        rec(f"gated delta: chunked scan ({kind}; {H} heads of {d} x {dv})",
+            timed(lambda: ops.gated_delta_scan(act, mats, proj, 0, plan, H, G, d, dv, taps, ring, memory, o)),
+            rows * (C + H * dv) * 4 + mats.numel() * 4 + state_bytes, delta_flops)
+    else:
+        rec(f"gated delta, one kernel: convolution to gated result ({kind}; {H} heads of {d} x {dv})",
+            timed(lambda: ops.gated_delta(proj, 0, a_off, b_off, g_off, plan, H, G, d, dv, conv_w, a_log, dt, d ** -0.5, 1e-6, norm_w, 1e-5,
+                                          ring, memory, mixed)), state_bytes + ring_bytes + rows * (proj.shape[1] * 4 + H * dv * 2), delta_flops)
+    turned = torch.empty(rows, C, device=dev)
+    rec("like: causal_conv with silu (the same channels)",
+        timed(lambda: ops.causal_conv(proj, 0, C, conv_w.to(bf), None, plan, cache.state[(0, "shift")], turned, act="silu")), rows * C * 8)
+    # the other delta rule at the same heads and state (every head with q, k and v of its own)
+    wide = torch.randn(rows, 5 * hk + 16, device=dev)
+    aux = torch.empty(rows, 3, hk, device=dev)
+    w2, w0 = torch.randn(hk, 16, device=dev).to(bf) * 0.1, torch.zeros(hk, device=dev, dtype=bf)
+    rec("like: delta_prep", timed(lambda: ops.delta_prep(wide, hk, 4 * hk, 5 * hk, H, d, w2, w0, w0, 0.6, 1e-6, aux)), rows * hk * 20)
+    if d == dv:
+        rec(f"like: delta_scan ({kind}; {H} heads of {d} x {d})",
+            timed(lambda: ops.delta_scan(wide, 0, hk, 2 * hk, aux, plan, H, d, memory, o)), rows * hk * 28 + state_bytes, delta_flops)
+    memory.zero_()
+    dec = torch.full((rows, H), 0.95, device=dev)
+    rec(f"like: linrec_scan, a decay per token and head ({kind}; {H} heads of {d} x {dv})",
+        timed(lambda: ops.linrec_scan(proj, 0, kw, 2 * kw, plan, H, d, dv, None, None, memory, o, token_decay=dec, heads_per_qk=H // G)),
+        rows * (C + H * dv) * 4 + state_bytes, lin_flops)
+    rec("linrec_out (norm and gate)", timed(lambda: ops.linrec_out(o, proj, g_off, H, dv, norm_w, 1e-5, mixed)), rows * H * dv * 10)
+    # attention beside it
+    store, g0 = cache.groups[0].entry_storage(0), plan.groups[0]
+    store.normal_()
+    aproj = torch.randn(rows, (2 * aH + 2 * aG) * ad, device=dev)
+    q = torch.randn(rows, aH, ad, device=dev).to(bf)
+    freq = frequency_table(2e5, ad // 2, dev)
+    hw = torch.ones(ad, device=dev, dtype=bf)
+    rec("attn_prep, every head normed before the rotation",
+        timed(lambda: ops.attn_prep(aproj, 0, 2 * aH * ad, (2 * aH + aG) * ad, aH, aG, ad, ad, ad, ad // 2, False, freq, None, hw, hw, 1e-5,
+                                    plan.row_seq, plan.row_pos, g0.page_off, g0.page_ids, g0.page_size, store, q, head_norm="before")),
+        rows * (aH + 2 * aG) * ad * 6)
+    fw, fk = torch.ones(aH * ad, device=dev, dtype=bf), torch.ones(aG * ad, device=dev, dtype=bf)
+    rec("like: attn_prep, whole projections normed",
+        timed(lambda: ops.attn_prep(aproj, 0, 2 * aH * ad, (2 * aH + aG) * ad, aH, aG, ad, ad, ad, ad // 2, False, freq, None, fw, fk, 1e-5,
+                                    plan.row_seq, plan.row_pos, g0.page_off, g0.page_ids, g0.page_size, store, q)),
+        rows * (aH + 2 * aG) * ad * 6)
+    q.normal_()
+    ao = torch.empty(rows, aH * ad, device=dev, dtype=bf)
+    keys = sum(min(i + 1, win) for i in range(rows)) if prompt else rows * min(past + 1, win)
+    rec(f"attention ({kind}; window {win})", timed(lambda: ops.attention(q, ao, plan, 0, store, aH, aG, ad, win, ad ** -0.5)),
+        (rows if prompt else keys) * aG * ad * 4 + rows * aH * ad * 4, 4 * keys * aH * ad)
+    both = torch.empty(rows, aH * ad + H * dv, device=dev, dtype=bf)
+    rec("attn_gate (a gate for every value, into the shared product's columns)",
+        timed(lambda: ops.attn_gate(ao, both, aH, ad, ad, (aproj, aH * ad), 0.9, 0)), rows * aH * ad * 8)
+    rec("like: attn_unrotate with a gate per head",
+        timed(lambda: ops.attn_unrotate(ao, both[:, :aH * ad].contiguous(), aH, ad, ad, False, None, plan.row_pos, gate=(aproj, 0))),
+        rows * aH * ad * 4)
+    # experts by token id
+    E, top, ff = moe["experts"], moe["top"], moe["expert_ff"]
+    etab = torch.stack([torch.randperm(E, generator=bench.gen)[:top] for _ in range(z["vocab"])]).int().to(dev)
+    rec("moe_group_by_token", timed(lambda: ops.moe_group_by_token(toks, etab, E, bf, ff, W)), rows * top * 16)
+    ids, order, meta = ops.moe_group_by_token(toks, etab, E, bf, ff, W)
+    logits, ids2, wts = torch.randn(rows, E, device=dev), torch.empty_like(ids), torch.empty(rows, top, device=dev)
+
+    def routed():
+        ops.moe_route_scored(logits, None, top, ids2, wts, scores="softmax", renormalize=True)
+        tile = int(ops.lib().sb_moe_tile_rows(1, rows * top, E, ff, W))
+        ops._check(ops.lib().sb_moe_group(ops._ptr(ids2), rows * top, E, tile, ops._ptr(order2), ops._ptr(meta2), ops._stream()), "moe_group")
+    order2, meta2 = torch.empty_like(order), torch.empty_like(meta)
+    rec("like: moe_route_scored, softmax, and moe_group", timed(routed), rows * (E * 4 + top * 24))
+    h = torch.randn(rows, W, device=dev).to(bf)
+    w1 = torch.randn(E, ff, W, device=dev, dtype=bf) * 0.02
+    w2e = torch.randn(E, W, ff, device=dev, dtype=bf) * 0.02
+    hit = len(set(ids.flatten().tolist()))
+    pairs = rows * top
+    rec("experts: up with squared relu, down", timed(lambda: ops._moe_pairs(h, ids, w1, w2e, ops.EXPERT_RELU2, 0.0, 0.0, (order, meta))),
+        hit * 2 * ff * W * 2 + rows * W * 2 + pairs * ff * 4 + pairs * W * 4, 4 * pairs * ff * W)
+    rec("like: experts: group, up with squared relu, down",
+        timed(lambda: ops._moe_pairs(h, ids, w1, w2e, ops.EXPERT_RELU2, 0.0, 0.0)),
+        hit * 2 * ff * W * 2 + rows * W * 2 + pairs * ff * 4 + pairs * W * 4, 4 * pairs * ff * W)
+    return out
+
+
+def run_sipilorn(args) -> int:
+    """Prefill and decode throughput of Sipilorn models at layer sizes of real models (random weights), with dense
+    feed-forwards beside the Mefupel models of equal width, depth, vocabulary, states, windows and feed-forward
+    values, and with experts by token id in every second layer; and each of its kernels alone beside the like
+    kernels of the other models."""
+    import torch
+    import sonicboom_b200 as sb
+    from sonicboom_b200 import ops
+
+    bench = ArchBench()
+    dev = bench.dev
+    result = {"arch": "sipilorn", "impl": "ours", "dtype": "bf16", "peaks": bench.pk, "sizes": {},
+              "data": "synthetic: random N(0,0.02) weights, uniform random token ids",
+              "timing": "CUDA events; kernels alone: median of 5 after 3 warm-up calls, L2 flushed "
+                        "(256 MB written) before each; models: prefill median of 3, decode one region of K steps"}
+    with ClockSampler() as clocks:
+        for name, z in SIPILORN_SIZES.items():
+            if args.sizes and name not in args.sizes.split(","):
+                continue
+            rec = {"sipilorn_config": dict(z, **SIPILORN_EXPERTS[name])}
+            for label, cfg in (("sipilorn, dense", sipilorn_config(**z)),
+                               ("mefupel (equal width, depth, vocab, states, windows, feed-forward values)", sipilorn_mefupel_config(z)),
+                               ("sipilorn, experts in every second layer", sipilorn_config(**z, **SIPILORN_EXPERTS[name]))):
+                m = sb.random_model(cfg, seed=0, dtype="bfloat16", device=dev, std=0.02)
+                rec[label] = bench.model_points(m, args.prompt, args.batch, args.steps, args.warmup)
+                del m
+                torch.cuda.empty_cache()
+            for rows in (args.prompt, args.batch):
+                rec["kernels_rows_%d" % rows] = sipilorn_kernels(bench, z, SIPILORN_EXPERTS[name], rows, args.prompt)
+            result["sizes"][name] = rec
+    ops.check_status()
+    result["clocks"] = clocks.summary()
+    print(json.dumps(result))
+    return 0
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1421,15 +1652,16 @@ def main() -> int:
                     help="run one phase only and print a short line (small cases for profilers)")
     ap.add_argument("--eager", action="store_true",
                     help="with --only decode: launch the step kernel by kernel, not as a graph")
-    ap.add_argument("--arch", choices=["qwen2", "zolulix", "mefupel", "leguvik", "bulodra", "debisun"], default="qwen2",
+    ap.add_argument("--arch", choices=["qwen2", "zolulix", "mefupel", "leguvik", "bulodra", "debisun", "sipilorn"], default="qwen2",
                     help="zolulix: that design's prefill and decode throughput and its kernels alone, "
                          "beside the Qwen2.5 decoder of equal sizes (its own JSON line; the default "
                          "workload is unchanged); mefupel: the same for that design, beside Zolulix and "
                          "Qwen2.5 models of equal sizes; leguvik: the same for that design, beside Mefupel "
                          "models of equal sizes; bulodra: the same for that design, beside Leguvik models of "
-                         "equal sizes; debisun: the same for that design, beside Bulodra models of equal sizes")
-    ap.add_argument("--sizes", default="", help="with --arch zolulix / mefupel / leguvik / bulodra / debisun: which of its sizes to run (comma separated)")
-    ap.add_argument("--prompt", type=int, default=2048, help="with --arch zolulix / mefupel / leguvik / bulodra / debisun: prompt length")
+                         "equal sizes; debisun: the same for that design, beside Bulodra models of equal sizes; "
+                         "sipilorn: the same for that design, beside Mefupel models of equal sizes")
+    ap.add_argument("--sizes", default="", help="with --arch zolulix / mefupel / leguvik / bulodra / debisun / sipilorn: which of its sizes to run (comma separated)")
+    ap.add_argument("--prompt", type=int, default=2048, help="with --arch zolulix / mefupel / leguvik / bulodra / debisun / sipilorn: prompt length")
     args = ap.parse_args()
     if args.impl == "reference":
         return reference_arm()
@@ -1448,6 +1680,8 @@ def main() -> int:
         return run_bulodra(args)
     if args.arch == "debisun":
         return run_debisun(args)
+    if args.arch == "sipilorn":
+        return run_sipilorn(args)
     return run(args)
 
 

@@ -421,8 +421,6 @@ def sharp_model():
 def sharpen(t):
     for n in t:
         if n.endswith(".o"):
-            t[n] *= 3.0
-        if n.endswith("q.norm") or n.endswith("k.norm"):
             t[n] *= 2.0
         if n.endswith("A_log"):
             t[n][:] = -7.0                             # every head remembers for long
