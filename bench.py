@@ -1514,7 +1514,7 @@ def sipilorn_kernels(bench, z, moe, rows, context):
         rec("gated delta: convolution, unit vectors, chunk matrices",
             timed(lambda: ops.gated_delta_prep(proj, 0, a_off, b_off, plan, H, G, d, dv, conv_w, a_log, dt, d ** -0.5, 1e-6, ring)),
             rows * C * 8 + mats.numel() * 4)
-        for cpt in (1, 2):
+        for cpt in (2, 4):
             ops.force_gated_delta_columns(cpt)
             rec(f"gated delta: chunked scan, {cpt} column(s) a thread ({kind}; {H} heads of {d} x {dv})",
                 timed(lambda: ops.gated_delta_scan(act, mats, proj, 0, plan, H, G, d, dv, taps, ring, memory, o)),

@@ -396,47 +396,81 @@ struct ScanArgs {
   float* out;                          // [rows, heads, vdim]
 };
 
-constexpr int SCAN_THREADS = 128, SCAN_GROUPS = SCAN_THREADS / LANES;
-constexpr int TP = TB + 4;                      // pitch of a staged matrix row: even rows first, then the odd ones
+constexpr int SCAN_THREADS = 128, SCAN_LANES = 16, SCAN_GROUPS = SCAN_THREADS / SCAN_LANES;
+constexpr int TP = TB + 4;                      // pitch of a staged matrix row
 constexpr int MAT_SM = 2 * TB * TP + 2 * TB;    // T, P, G, D_15
+constexpr int HALF = TB / 2;
 
 template <int NPL, int CPT>
 struct ScanShape {
-  static constexpr int PAD = NPL * LANES, COLS = SCAN_GROUPS * CPT;
-  static constexpr int STAGE = 2 * TB * PAD + TB * COLS + MAT_SM;       // q, k, values, matrices
-  static constexpr int XP = TB + 4;                                     // pitch of a group's exchange buffer
+  static constexpr int PAD = NPL * SCAN_LANES, COLS = SCAN_GROUPS * CPT;
+  static constexpr int VP = COLS + 4;                                   // pitch of a token's values
+  static constexpr int STAGE = 2 * TB * PAD + TB * VP + MAT_SM;         // q, k, values, matrices
+  static constexpr int XP = TB + 4;                                     // pitch of a column's exchange buffer
   static constexpr int EXTRA = SCAN_GROUPS * CPT * XP;
   static constexpr size_t bytes(int stages) { return ((size_t)stages * STAGE + EXTRA) * sizeof(float); }
 };
 
-// The LANES lanes of a column add their parts of 16 tokens' sums, halving what a lane keeps each time: lane `sub` ends
-// with the sums of tokens 2 sub and 2 sub + 1, by the same tree of additions for every token.
-__device__ __forceinline__ void share_sums(float (&a)[TB], int sub, float& s0, float& s1) {
+template <int N>
+struct Size {
+  static constexpr int value = N;
+};
+
+// Two float32 values side by side: one fma instruction works on both, each rounded as a fma of its own.
+struct Two {
+  unsigned long long v;
+};
+__device__ __forceinline__ Two two(float lo, float hi) {
+  Two r;
+  asm("mov.b64 %0, {%1, %2};\n" : "=l"(r.v) : "f"(lo), "f"(hi));
+  return r;
+}
+__device__ __forceinline__ float2 parts(Two a) {
+  float2 r;
+  asm("mov.b64 {%0, %1}, %2;\n" : "=f"(r.x), "=f"(r.y) : "l"(a.v));
+  return r;
+}
+__device__ __forceinline__ Two fma2(Two a, Two b, Two c) {
+  Two r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;\n" : "=l"(r.v) : "l"(a.v), "l"(b.v), "l"(c.v));
+  return r;
+}
+
+// The lanes of a column add their parts of eight tokens' sums, halving what a lane keeps each time: lane `sub` ends with the
+// sum of token sub % 8, by the same tree of additions for every token.
+__device__ __forceinline__ float share_sums(float (&a)[HALF], int sub) {
 #pragma unroll
-  for (int w = LANES / 2, n = TB / 2; w > 0; w >>= 1, n >>= 1) {
+  for (int w = HALF / 2; w > 0; w >>= 1) {
     const bool up = sub & w;
 #pragma unroll
-    for (int i = 0; i < n; ++i) {
-      const float keep = up ? a[i + n] : a[i], give = up ? a[i] : a[i + n];
+    for (int i = 0; i < w; ++i) {
+      const float keep = up ? a[i + w] : a[i], give = up ? a[i] : a[i + w];
       a[i] = keep + __shfl_xor_sync(0xffffffffu, give, w);
     }
   }
-  s0 = a[0];
-  s1 = a[1];
+  return a[0] + __shfl_xor_sync(0xffffffffu, a[0], HALF);
 }
 
+// A lane keeps NPL channels (in pairs) of CPT neighbouring columns for the whole step: what it reads of a token's q
+// and k from shared memory serves CPT columns, and shared memory's bandwidth, a value a lane and cycle, is what
+// the kernel runs against.  With up to 8 channels a lane also keeps the chunk's keys in registers from the first pass (S^T k)
+// to the last (the update).
 template <int NPL, int CPT, bool VEC, int STAGES>
 __global__ void __launch_bounds__(SCAN_THREADS) gdelta_scan_kernel(const ScanArgs p) {
   using Sh = ScanShape<NPL, CPT>;
-  constexpr int PAD = Sh::PAD, COLS = Sh::COLS, R = Runs<NPL>::R, V = VEC ? 4 : 1;
+  constexpr int PAD = Sh::PAD, COLS = Sh::COLS, V = VEC ? 4 : 1;
+  constexpr int R = NPL < 4 ? NPL : 4, N2 = NPL / 2;      // values of a run; pairs of a lane
+  constexpr bool KEEP = NPL <= 8;
   extern __shared__ __align__(16) float sm[];
   float* xbuf = sm + STAGES * Sh::STAGE;
   sb_pdl_launch();
-  const int b = blockIdx.z, h = blockIdx.y, tid = threadIdx.x, sub = tid % LANES, cl = tid / LANES;
+  const int b = blockIdx.z, h = blockIdx.y, tid = threadIdx.x, sub = tid % SCAN_LANES, cl = tid / SCAN_LANES;
   const int dim = p.dim, vdim = p.vdim, taps = p.taps, per = p.n_heads / p.n_kv_heads, kv = h / per;
   const int kw = p.n_kv_heads * dim, C = 2 * kw + p.n_heads * vdim;
   const int col0 = blockIdx.x * COLS, col = col0 + cl * CPT;
   const int row0 = p.seq_row0[b], n = p.seq_row0[b + 1] - row0, slot = p.seq_slot[b];
+  // lane `sub`'s channel i: runs of R, as far apart as the lanes' runs are long together
+  auto channel = [&](int i) { return (i / R) * (SCAN_LANES * R) + sub * R + i % R; };
   if (PAD > dim || vdim - col0 < COLS) {          // channels and columns past the sizes stay zero for good
     for (int i = tid; i < STAGES * Sh::STAGE; i += SCAN_THREADS) sm[i] = 0.0f;
     __syncthreads();
@@ -444,32 +478,39 @@ __global__ void __launch_bounds__(SCAN_THREADS) gdelta_scan_kernel(const ScanArg
   sb_pdl_wait();
   const float* act = p.act + (size_t)row0 * C;
   const float* mats = p.mats + ((size_t)chunk_base(row0, b) * p.n_heads + h) * MATS;
-  // a thread keeps to pieces tid % W, + W, ... of a row and takes tokens tid / W, + THREADS / W, ...
+  // Staging: a thread keeps to its pieces (V values) of a token's row and takes tokens STEP apart; every division is by a
+  // constant, and a chunk's source addresses follow from the first one's.
   const int n_vals = min(COLS, vdim - col0);
+  auto copy = [&](float* to, int pitch, const float* from, int t0, int width, auto padded) {   // `width` values of 16 tokens' rows
+    constexpr int PIECES = decltype(padded)::value / V, W = PIECES < SCAN_THREADS ? PIECES : SCAN_THREADS, STEP = SCAN_THREADS / W;
+    const int first = tid / W, piece = tid % W;
+    if (W * STEP < SCAN_THREADS && first >= STEP) return;
+#pragma unroll
+    for (int t = first; t < TB; t += STEP) {
+      const bool ok = t0 + t < n;
+      const float* row = ok ? from + (size_t)(t0 + t) * C : act;
+#pragma unroll
+      for (int i = piece; i < PIECES; i += W)
+        if (i * V < width) {
+          if (VEC) cp_async16(to + t * pitch + i * V, row + (ok ? i * V : 0), ok);
+          else cp_async4(to + t * pitch + i, row + (ok ? i : 0), ok);
+        }
+    }
+  };
+  const float* q_src = act + kv * dim;
+  const float* k_src = q_src + kw;
+  const float* v_src = act + 2 * kw + h * vdim + col0;
   auto stage = [&](int st, int ch) {
     float* dst = sm + (size_t)st * Sh::STAGE;
-    const int t0 = ch * TB;
-    auto copy = [&](float* to, int pitch, const float* from, int width) {      // `width` values of 16 tokens' rows of act
-      const int pieces = (width + V - 1) / V, W = pieces < SCAN_THREADS ? pieces : SCAN_THREADS, step = SCAN_THREADS / W;
-      if (tid >= W * step) return;
-      for (int t = tid / W; t < TB; t += step)
-        for (int i = tid % W; i < pieces; i += W) {
-          const bool ok = t0 + t < n;
-          const float* src = ok ? from + (size_t)(t0 + t) * C + i * V : act;
-          if (VEC) cp_async16(to + t * pitch + i * V, src, ok);
-          else cp_async4(to + t * pitch + i, src, ok);
-        }
-    };
-    copy(dst, PAD, act + kv * dim, dim);
-    copy(dst + TB * PAD, PAD, act + kw + kv * dim, dim);
-    copy(dst + 2 * TB * PAD, COLS, act + 2 * kw + h * vdim + col0, n_vals);
-    float* m = dst + 2 * TB * PAD + TB * COLS;
+    copy(dst, PAD, q_src, ch * TB, dim, Size<PAD>());
+    copy(dst + TB * PAD, PAD, k_src, ch * TB, dim, Size<PAD>());
+    copy(dst + 2 * TB * PAD, Sh::VP, v_src, ch * TB, n_vals, Size<COLS>());
+    float* m = dst + 2 * TB * PAD + TB * Sh::VP;
     const float* src = mats + (size_t)ch * p.n_heads * MATS;
+#pragma unroll
     for (int i = tid; i < MATS / 4; i += SCAN_THREADS) {
-      const int e = i * 4, r = (e / TB) % TB;                                     // row of T or P
-      const int at = e < 2 * TB * TB ? (e / (TB * TB)) * TB * TP + ((r & 1) * (TB / 2) + (r >> 1)) * TP + e % TB
-                                     : 2 * TB * TP + e - 2 * TB * TB;
-      cp_async16(m + at, src + e, true);
+      const int e = i * 4;
+      cp_async16(m + (e < 2 * TB * TB ? (e / TB) * TP + e % TB : 2 * TB * TP + e - 2 * TB * TB), src + e, true);
     }
   };
   const int n_chunks = (n + TB - 1) / TB;
@@ -479,15 +520,34 @@ __global__ void __launch_bounds__(SCAN_THREADS) gdelta_scan_kernel(const ScanArg
     cp_commit();
   }
   float* memory = p.memory + ((size_t)slot * p.n_heads + h) * vdim * dim;
-  float S[CPT][NPL];
+  Two S[CPT][N2];
 #pragma unroll
   for (int x = 0; x < CPT; ++x)
 #pragma unroll
-    for (int i = 0; i < NPL; ++i) {
-      const int c = Runs<NPL>::channel(sub, i);
-      S[x][i] = col + x < vdim && c < dim ? memory[(size_t)(col + x) * dim + c] : 0.0f;
+    for (int i = 0; i < N2; ++i) {
+      float v[2];
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int c = channel(2 * i + e);
+        v[e] = col + x < vdim && c < dim ? memory[(size_t)(col + x) * dim + c] : 0.0f;
+      }
+      S[x][i] = two(v[0], v[1]);
     }
   float* xb = xbuf + cl * CPT * Sh::XP;
+  auto load_row = [&](const float* row, Two (&r)[N2]) {   // this lane's channels of a token's q or k
+#pragma unroll
+    for (int j = 0; j < NPL / R; ++j) {
+      const float* at = row + j * (SCAN_LANES * R) + sub * R;
+      if constexpr (R == 4) {
+        const float4 f = *reinterpret_cast<const float4*>(at);
+        r[2 * j] = two(f.x, f.y);
+        r[2 * j + 1] = two(f.z, f.w);
+      } else {
+        const float2 f = *reinterpret_cast<const float2*>(at);
+        r[j] = two(f.x, f.y);
+      }
+    }
+  };
 
   for (int ch = 0; ch < n_chunks; ++ch) {
     cp_wait<STAGES - 2>();
@@ -497,126 +557,125 @@ __global__ void __launch_bounds__(SCAN_THREADS) gdelta_scan_kernel(const ScanArg
     const float* q = sm + (size_t)(ch % STAGES) * Sh::STAGE;
     const float* k = q + TB * PAD;
     const float* v = k + TB * PAD;
-    const float* T = v + TB * COLS;
+    const float* T = v + TB * Sh::VP;
     const float* P = T + TB * TP;
     const float* G = P + TB * TP;
     const float* D = G + TB;
-    // S^T k_t (or S^T q_t) of the chunk's tokens; this lane ends with those of tokens 2 sub, 2 sub + 1
-    auto project = [&](const float* rows, float (&s0)[CPT], float (&s1)[CPT]) {
-      float acc[CPT][TB];
+    Two kr[KEEP ? TB : 1][N2];
+    // S^T k_t and S^T q_t of the chunk's tokens: lane `sub` ends with those of token `sub`
+    float d[CPT], o[CPT];
 #pragma unroll
-      for (int t = 0; t < TB; ++t) {
+    for (int pass = 0; pass < 2; ++pass)
 #pragma unroll
-        for (int x = 0; x < CPT; ++x) acc[x][t] = 0.0f;
+      for (int half = 0; half < 2; ++half) {
+        float acc[CPT][HALF];
 #pragma unroll
-        for (int jj = 0; jj < NPL / R; ++jj) {
-          float r[R];
-          const float* at = rows + t * PAD + jj * (LANES * R) + sub * R;
-          if (R == 4) {
-            const float4 f = *reinterpret_cast<const float4*>(at);
-            r[0] = f.x; r[1 % R] = f.y; r[2 % R] = f.z; r[3 % R] = f.w;
-          } else {
+        for (int t = 0; t < HALF; ++t) {
+          Two r[N2];
+          load_row((pass == 0 ? k : q) + (half * HALF + t) * PAD, r);
 #pragma unroll
-            for (int e = 0; e < R; ++e) r[e] = at[e];
+          for (int x = 0; x < CPT; ++x) {
+            Two a = two(0.0f, 0.0f);
+#pragma unroll
+            for (int i = 0; i < N2; ++i) a = fma2(r[i], S[x][i], a);
+            const float2 f = parts(a);
+            acc[x][t] = f.x + f.y;
           }
+          if (KEEP && pass == 0)
 #pragma unroll
-          for (int x = 0; x < CPT; ++x)
+            for (int i = 0; i < N2; ++i) kr[half * HALF + t][i] = r[i];
+        }
 #pragma unroll
-            for (int e = 0; e < R; ++e) acc[x][t] = fmaf(r[e], S[x][jj * R + e], acc[x][t]);
+        for (int x = 0; x < CPT; ++x) {
+          const float y = share_sums(acc[x], sub);
+          if (half == 0 || (sub & HALF)) (pass == 0 ? d : o)[x] = y;
         }
       }
+    // w = v - G * (S^T k), to the column's other lanes; u = T w
+    const float g_own = G[sub], g_all = G[TB - 1];
+    float own[CPT];
+    if constexpr (CPT == 4) {
+      const float4 f = *reinterpret_cast<const float4*>(v + sub * Sh::VP + cl * CPT);
+      own[0] = f.x; own[1] = f.y; own[2] = f.z; own[3] = f.w;
+    } else {
 #pragma unroll
-      for (int x = 0; x < CPT; ++x) share_sums(acc[x], sub, s0[x], s1[x]);
-    };
-    // y = the 16 tokens' values of a column from the lanes' pairs
-    auto gather = [&](const float (&a0)[CPT], const float (&a1)[CPT], float (&y)[CPT][TB]) {
-      __syncwarp();
-#pragma unroll
-      for (int x = 0; x < CPT; ++x) *reinterpret_cast<float2*>(xb + x * Sh::XP + 2 * sub) = make_float2(a0[x], a1[x]);
-      __syncwarp();
-#pragma unroll
-      for (int x = 0; x < CPT; ++x)
-#pragma unroll
-        for (int i = 0; i < TB; i += 4) {
-          const float4 f = *reinterpret_cast<const float4*>(xb + x * Sh::XP + i);
-          y[x][i] = f.x; y[x][i + 1] = f.y; y[x][i + 2] = f.z; y[x][i + 3] = f.w;
-        }
-    };
-    // row 2 sub (first half) or 2 sub + 1 (second half) of a matrix times y
-    auto row_dot = [&](const float* m, int half, const float (&y)[TB]) {
-      const float* r = m + (half * (TB / 2) + sub) * TP;
-      float s = 0.0f;
-#pragma unroll
-      for (int i = 0; i < TB; i += 4) {
-        const float4 f = *reinterpret_cast<const float4*>(r + i);
-        s = fmaf(f.x, y[i], s); s = fmaf(f.y, y[i + 1], s); s = fmaf(f.z, y[i + 2], s); s = fmaf(f.w, y[i + 3], s);
-      }
-      return s;
-    };
-    float d0[CPT], d1[CPT], o0[CPT], o1[CPT];
-    project(k, d0, d1);
-    project(q, o0, o1);
-    const float g0 = G[2 * sub], g1 = G[2 * sub + 1], g_all = G[TB - 1];
-#pragma unroll
-    for (int x = 0; x < CPT; ++x) {
-      d0[x] = v[(2 * sub) * COLS + cl * CPT + x] - g0 * d0[x];
-      d1[x] = v[(2 * sub + 1) * COLS + cl * CPT + x] - g1 * d1[x];
+      for (int x = 0; x < CPT; ++x) own[x] = v[sub * Sh::VP + cl * CPT + x];
     }
-    float u[CPT][TB];
-    gather(d0, d1, u);
+    __syncwarp();
 #pragma unroll
-    for (int x = 0; x < CPT; ++x) {
-      d0[x] = row_dot(T, 0, u[x]);
-      d1[x] = row_dot(T, 1, u[x]);
-    }
-    gather(d0, d1, u);
+    for (int x = 0; x < CPT; ++x) xb[x * Sh::XP + sub] = own[x] - g_own * d[x];
+    __syncwarp();
 #pragma unroll
-    for (int x = 0; x < CPT; ++x) {
-      o0[x] = fmaf(g0, o0[x], row_dot(P, 0, u[x]));
-      o1[x] = fmaf(g1, o1[x], row_dot(P, 1, u[x]));
-      if (col + x < vdim) {
-        const int t = ch * TB + 2 * sub;
-        float* o = p.out + ((size_t)(row0 + t) * p.n_heads + h) * vdim + col + x;
-        if (t < n) o[0] = o0[x];
-        if (t + 1 < n) o[(size_t)p.n_heads * vdim] = o1[x];
-      }
-    }
+    for (int x = 0; x < CPT; ++x) d[x] = 0.0f, o[x] *= g_own;
 #pragma unroll
     for (int i = 0; i < TB; i += 4) {
-      const float4 f = *reinterpret_cast<const float4*>(D + i);
+      const float4 m = *reinterpret_cast<const float4*>(T + sub * TP + i);
 #pragma unroll
-      for (int x = 0; x < CPT; ++x) u[x][i] *= f.x, u[x][i + 1] *= f.y, u[x][i + 2] *= f.z, u[x][i + 3] *= f.w;
+      for (int x = 0; x < CPT; ++x) {
+        const float4 w = *reinterpret_cast<const float4*>(xb + x * Sh::XP + i);
+        d[x] = fmaf(m.x, w.x, d[x]); d[x] = fmaf(m.y, w.y, d[x]); d[x] = fmaf(m.z, w.z, d[x]); d[x] = fmaf(m.w, w.w, d[x]);
+      }
     }
+    __syncwarp();
+#pragma unroll
+    for (int x = 0; x < CPT; ++x) xb[x * Sh::XP + sub] = d[x];
+    __syncwarp();
+    const Two gg = two(g_all, g_all), zero = two(0.0f, 0.0f);
 #pragma unroll
     for (int x = 0; x < CPT; ++x)
 #pragma unroll
-      for (int i = 0; i < NPL; ++i) S[x][i] *= g_all;
+      for (int i = 0; i < N2; ++i) S[x][i] = fma2(S[x][i], gg, zero);
+    // o += P u;  S += sum_j D_15,j k_j u_j
 #pragma unroll
-    for (int t = 0; t < TB; ++t)
+    for (int i = 0; i < TB; i += 4) {
+      const float4 m = *reinterpret_cast<const float4*>(P + sub * TP + i), f = *reinterpret_cast<const float4*>(D + i);
+      const float dd[4] = {f.x, f.y, f.z, f.w};
+      float u[CPT][4];
 #pragma unroll
-      for (int jj = 0; jj < NPL / R; ++jj) {
-        float r[R];
-        const float* at = k + t * PAD + jj * (LANES * R) + sub * R;
-        if (R == 4) {
-          const float4 f = *reinterpret_cast<const float4*>(at);
-          r[0] = f.x; r[1 % R] = f.y; r[2 % R] = f.z; r[3 % R] = f.w;
+      for (int x = 0; x < CPT; ++x) {
+        const float4 w = *reinterpret_cast<const float4*>(xb + x * Sh::XP + i);
+        o[x] = fmaf(m.x, w.x, o[x]); o[x] = fmaf(m.y, w.y, o[x]); o[x] = fmaf(m.z, w.z, o[x]); o[x] = fmaf(m.w, w.w, o[x]);
+        u[x][0] = w.x; u[x][1] = w.y; u[x][2] = w.z; u[x][3] = w.w;
+      }
+#pragma unroll
+      for (int t = 0; t < 4; ++t) {
+        Two r[N2];
+        if (KEEP) {
+#pragma unroll
+          for (int e = 0; e < N2; ++e) r[e] = kr[KEEP ? i + t : 0][e];
         } else {
-#pragma unroll
-          for (int e = 0; e < R; ++e) r[e] = at[e];
+          load_row(k + (i + t) * PAD, r);
         }
 #pragma unroll
-        for (int x = 0; x < CPT; ++x)
+        for (int x = 0; x < CPT; ++x) {
+          const float e = dd[t] * u[x][t];
+          const Two ee = two(e, e);
 #pragma unroll
-          for (int e = 0; e < R; ++e) S[x][jj * R + e] = fmaf(r[e], u[x][t], S[x][jj * R + e]);
+          for (int j = 0; j < N2; ++j) S[x][j] = fma2(r[j], ee, S[x][j]);
+        }
       }
+    }
+    const int t = ch * TB + sub;
+    if (t < n) {
+      float* to = p.out + ((size_t)(row0 + t) * p.n_heads + h) * vdim + col;
+      if (VEC && CPT == 4) {            // vdim is a multiple of four, so four columns are all there or none is
+        if (col < vdim) *reinterpret_cast<float4*>(to) = make_float4(o[0], o[1 % CPT], o[2 % CPT], o[3 % CPT]);
+      } else {
+#pragma unroll
+        for (int x = 0; x < CPT; ++x)
+          if (col + x < vdim) to[x] = o[x];
+      }
+    }
   }
   cp_wait<0>();
 #pragma unroll
   for (int x = 0; x < CPT; ++x)
 #pragma unroll
-    for (int i = 0; i < NPL; ++i) {
-      const int c = Runs<NPL>::channel(sub, i);
-      if (col + x < vdim && c < dim) memory[(size_t)(col + x) * dim + c] = S[x][i];
+    for (int i = 0; i < N2; ++i) {
+      const float2 f = parts(S[x][i]);
+      const int c = channel(2 * i);
+      if (col + x < vdim && c < dim) memory[(size_t)(col + x) * dim + c] = f.x;
+      if (col + x < vdim && c + 1 < dim) memory[(size_t)(col + x) * dim + c + 1] = f.y;
     }
   // the convolution's last inputs (the kernel before this one has read the old ones): a head keeps its own values'
   // channels, a group's first head those of q and k too
@@ -640,8 +699,9 @@ int sm_count() {
   return n;
 }
 
-template <int NPL, int CPT, bool VEC, int STAGES>
-cudaError_t launch_scan_staged(const ScanArgs& a, int n_seqs, cudaStream_t stream) {
+template <int NPL, int CPT, bool VEC>
+cudaError_t launch_scan_columns(const ScanArgs& a, int n_seqs, cudaStream_t stream) {
+  constexpr int STAGES = ScanShape<NPL, CPT>::bytes(3) <= 112 * 1024 ? 3 : 2;
   constexpr size_t smem = ScanShape<NPL, CPT>::bytes(STAGES);
   static bool configured = false;
   if (!configured && smem > 48 * 1024) {
@@ -655,16 +715,20 @@ cudaError_t launch_scan_staged(const ScanArgs& a, int n_seqs, cudaStream_t strea
 
 int g_force_cpt = 0;
 
-// Two columns a thread where that still gives every SM blocks enough, else one; three stages where they fit a block.
+// Four columns a thread where that still gives every SM a block, else two; the largest key sizes keep fewer.  Measured on
+// B200, 2,048 tokens of one sequence, heads of 128 x 128: 56 heads (224 blocks of four columns a thread) 525 us against
+// 603 us with two, 32 heads (128 blocks) 325 against 312 us, 16 heads 324 against 202 us.
 template <int NPL, bool VEC>
 cudaError_t launch_scan(const ScanArgs& a, int n_seqs, cudaStream_t stream) {
-  constexpr int STAGES = ScanShape<NPL, 2>::bytes(3) <= 112 * 1024 ? 3 : 2;
-  if constexpr (NPL <= 16) {
-    const long blocks2 = (long)((a.vdim + 2 * SCAN_GROUPS - 1) / (2 * SCAN_GROUPS)) * a.n_heads * n_seqs;
-    if (g_force_cpt ? g_force_cpt == 2 : blocks2 >= 3L * sm_count())
-      return launch_scan_staged<NPL, 2, VEC, STAGES>(a, n_seqs, stream);
+  if constexpr (NPL > 16) {
+    return launch_scan_columns<NPL, 1, VEC>(a, n_seqs, stream);
+  } else if constexpr (NPL > 8 || !VEC) {
+    return launch_scan_columns<NPL, 2, VEC>(a, n_seqs, stream);
+  } else {
+    const long blocks4 = (long)((a.vdim + 4 * SCAN_GROUPS - 1) / (4 * SCAN_GROUPS)) * a.n_heads * n_seqs;
+    if (g_force_cpt ? g_force_cpt == 4 : blocks4 >= sm_count()) return launch_scan_columns<NPL, 4, VEC>(a, n_seqs, stream);
+    return launch_scan_columns<NPL, 2, VEC>(a, n_seqs, stream);
   }
-  return launch_scan_staged<NPL, 1, VEC, STAGES>(a, n_seqs, stream);
 }
 
 int check_sizes(const char* what, int n_heads, int n_kv_heads, int dim, int vdim, int taps) {
@@ -774,20 +838,19 @@ extern "C" int sb_gdelta_scan(const float* act, const float* mats, const float* 
   a.act = act; a.mats = mats; a.proj = proj; a.ld = ld; a.q_off = q_off; a.n_heads = n_heads; a.n_kv_heads = n_kv_heads;
   a.dim = dim; a.vdim = vdim; a.taps = taps; a.seq_row0 = seq_row0; a.seq_pos0 = seq_pos0; a.seq_slot = seq_slot;
   a.ring = taps > 1 ? ring : nullptr; a.memory = memory; a.out = out;
-  const bool vec = dim % 4 == 0 && vdim % 4 == 0 && !((uintptr_t)act & 15);
-  const int need = (dim + LANES - 1) / LANES;
+  const bool vec = dim % 4 == 0 && vdim % 4 == 0 && !(((uintptr_t)act | (uintptr_t)out) & 15);
+  const int need = (dim + SCAN_LANES - 1) / SCAN_LANES;
   cudaError_t e;
 #define SB_GD_SCAN(N) e = vec ? launch_scan<N, true>(a, n_seqs, stream) : launch_scan<N, false>(a, n_seqs, stream)
   if (need <= 2) SB_GD_SCAN(2);
   else if (need <= 4) SB_GD_SCAN(4);
   else if (need <= 8) SB_GD_SCAN(8);
   else if (need <= 16) SB_GD_SCAN(16);
-  else if (need <= 32) SB_GD_SCAN(32);
-  else SB_GD_SCAN(64);
+  else SB_GD_SCAN(32);
 #undef SB_GD_SCAN
   if (e != cudaSuccess) SB_FAIL(SB_ERR_CUDA, "sb_gdelta_scan: launch failed: %s", cudaGetErrorString(e));
   return SB_OK;
 }
 
-// For measurements and tests: 1 or 2 columns per thread for every call (where the key size allows two), 0 by the sizes again.
-extern "C" void sb_gdelta_force_columns(int cpt) { g_force_cpt = cpt == 1 || cpt == 2 ? cpt : 0; }
+// For measurements and tests: 2 or 4 columns per thread for every call (where the sizes allow four), 0 by the sizes again.
+extern "C" void sb_gdelta_force_columns(int cpt) { g_force_cpt = cpt == 2 || cpt == 4 ? cpt : 0; }

@@ -385,7 +385,7 @@ int sb_gdelta_scan(const float* act, const float* mats, const float* proj, int l
                    int n_kv_heads, int dim, int vdim, int taps, int n_seqs, const int32_t* seq_row0,
                    const int32_t* seq_pos0, const int32_t* seq_slot, float* ring, float* memory, float* out,
                    sb_stream_t stream);
-void sb_gdelta_force_columns(int cpt);   /* 1 or 2 columns per thread in sb_gdelta_scan; 0: by the sizes */
+void sb_gdelta_force_columns(int cpt);   /* 2 or 4 columns per thread in sb_gdelta_scan; 0: by the sizes */
 
 /* ---- the state-space mixer's rows ----
  * decay [rows, n_heads] = exp(-exp(a_log) dt), dt = softplus(proj[dt_off + h] + dt_bias); the row

@@ -1242,8 +1242,8 @@ def gated_delta_scan(act, mats, proj, q_off, plan, n_heads, n_kv_heads, dim, vdi
 
 
 def force_gated_delta_columns(cpt: int) -> None:
-    """1 or 2: every chunked scan of the gated delta rule keeps that many columns of the state per thread where the
-    key size allows it (for measurements and tests); 0: chosen by the sizes again."""
+    """2 or 4: every chunked scan of the gated delta rule keeps that many columns of the state per thread where the
+    sizes allow it (for measurements and tests); 0: chosen by the sizes again."""
     lib().sb_gdelta_force_columns(int(cpt))
 
 
